@@ -106,6 +106,10 @@ class ModelSpec:
     #: output, in 32-bit), with its tensor-name prefix; None: the embedding as it is
     embed_norm: PartSpec | None = None
     embed_norm_name: str = ""
+    #: something the embedding adds to the tokens' own vectors (a key of TOKEN_EMBEDDINGS with its
+    #: sizes), with its tensor-name prefix; None: the tokens' vectors alone
+    token_embedding: PartSpec | None = None
+    token_embedding_name: str = ""
 
     def __post_init__(self) -> None:
         if self.position_sinusoid_base < 0:

@@ -30,7 +30,8 @@ namespace sllm {
 
 // a: [N, lda] with the query latent at column 0 (Rq entries) and the key/value latent at column
 // kv_col (R entries) followed by the shared key part (r entries).  Two blocks per token: grid
-// (N, 2), one for the query latent and one for what is stored.
+// (N, 2), one for the query latent and one for what is stored; Rq 0 (queries without a latent):
+// grid (N, 1), only what is stored.
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_prep_kernel(const T* __restrict__ a, int64_t lda, int Rq, int kv_col, int R, int r,
@@ -45,7 +46,8 @@ latent_prep_kernel(const T* __restrict__ a, int64_t lda, int Rq, int kv_col, int
     const int64_t n = blockIdx.x;
     const T* row = a + n * lda;
     float ss = 0.f;
-    if (blockIdx.y == 0 && vec) {      // the query latent with 16-byte accesses
+    const int part = Rq > 0 ? blockIdx.y : 1;
+    if (part == 0 && vec) {            // the query latent with 16-byte accesses
         constexpr int VN = Vec<T>::N;
         float first[VN];               // a thread's first vector stays in registers
         for (int e = threadIdx.x * VN; e < Rq; e += blockDim.x * VN) {
@@ -79,7 +81,7 @@ latent_prep_kernel(const T* __restrict__ a, int64_t lda, int Rq, int kv_col, int
         }
         return;
     }
-    if (blockIdx.y == 0) {             // the query latent; the other block of the token stores
+    if (part == 0) {                   // the query latent; the other block of the token stores
         for (int e = threadIdx.x; e < Rq; e += blockDim.x) {
             const float v = to_float(row[e]);
             ss = fmaf(v, v, ss);
@@ -287,7 +289,7 @@ latent_q_rot_vec_kernel(const T* __restrict__ q, int64_t ldq, int H, int d, int 
 // output meet in shared memory and are added in the order of the warps, so a token's result
 // depends on nothing else in the batch.  The matrices of a step are small (H K J entries), so
 // what counts is that enough CTAs have enough loads in flight.  Options: `gate` (f = sigmoid of
-// gate[n * ldg + h], else 1), and a rotated tail as latent_q_rot_kernel writes it (the head's
+// gate[n * ldg + h], or with gate_wide of gate[n * ldg + h * J + j]; else 1), and a rotated tail as latent_q_rot_kernel writes it (the head's
 // entries K .. K + r of x, rotated, at out columns J .. J + tail, zeros behind the r), which the
 // CTAs of the first outputs write.
 constexpr int LS_T = 8;
@@ -298,7 +300,7 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 latent_small_kernel(const T* __restrict__ x, int64_t ldx, int64_t hsx, const T* __restrict__ w,
                     T* __restrict__ out, int64_t ldo, int64_t hso, int N, int K, int J,
-                    const T* __restrict__ gate, int64_t ldg, int r, int tail,
+                    const T* __restrict__ gate, int64_t ldg, int gate_wide, int r, int tail,
                     const int* __restrict__ positions, const float* __restrict__ cos_t,
                     const float* __restrict__ sin_t, int rot_dims) {
     extern __shared__ float ls_smem[];
@@ -354,7 +356,9 @@ latent_small_kernel(const T* __restrict__ x, int64_t ldx, int64_t hsx, const T* 
         for (int gg = 1; gg < LS_G; ++gg) sum += red[(gg * LS_T + t) * LS_J + lane];
         if (t < nt && j < J) {
             float f = 1.f;
-            if (gate) f = 1.0f / (1.0f + expf(-to_float(gate[(int64_t)(n0 + t) * ldg + h])));
+            if (gate)
+                f = 1.0f / (1.0f + expf(-to_float(gate[(int64_t)(n0 + t) * ldg +
+                                                       (gate_wide ? h * J + j : h)])));
             out[(int64_t)(n0 + t) * ldo + h * hso + j] = from_float<T>(sum * f);
         }
     }
@@ -389,21 +393,21 @@ SLLM_EXPORT int sllm_latent_prep(const void* a, int64_t lda, int Rq, int kv_col,
                                  const int* block_table, int table_stride, int page_size, int Dp,
                                  int write, int n_tokens, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (Rq < 1 || R < 1 || r < 0 || rot_dims < 0 || (rot_dims & 1) || rot_dims > r ||
+    if (Rq < 0 || R < 1 || r < 0 || rot_dims < 0 || (rot_dims & 1) || rot_dims > r ||
         Dp < R + r || page_size < 1 || kv_col < 0)
         return (int)cudaErrorInvalidValue;
     typedef __nv_bfloat16 bf16;
     // the query latent moves 16 bytes at a time where its rows allow it
     const int vn = dtype == 0 ? 4 : 8;
-    const int vec = Rq % vn == 0 && lda % vn == 0 &&
+    const int vec = Rq > 0 && Rq % vn == 0 && lda % vn == 0 &&
                     !(((uintptr_t)a | (uintptr_t)cq | (uintptr_t)q_gain) & 15);
     if (dtype == 0)
-        return (int)sllm_launch_pdl(latent_prep_kernel<float>, dim3(n_tokens, 2), dim3(256), 0, stream,
+        return (int)sllm_launch_pdl(latent_prep_kernel<float>, dim3(n_tokens, Rq > 0 ? 2 : 1), dim3(256), 0, stream,
                                     (const float*)a, lda, Rq, kv_col, R, r, q_gain, kv_gain, eps,
                                     positions, token_row, cos_t, sin_t, rot_dims, (float*)cq,
                                     (float*)pages, block_table, table_stride, page_size, Dp, write, vec);
     if (dtype == 1)
-        return (int)sllm_launch_pdl(latent_prep_kernel<bf16>, dim3(n_tokens, 2), dim3(256), 0, stream,
+        return (int)sllm_launch_pdl(latent_prep_kernel<bf16>, dim3(n_tokens, Rq > 0 ? 2 : 1), dim3(256), 0, stream,
                                     (const bf16*)a, lda, Rq, kv_col, R, r, q_gain, kv_gain, eps,
                                     positions, token_row, cos_t, sin_t, rot_dims, (bf16*)cq,
                                     (bf16*)pages, block_table, table_stride, page_size, Dp, write, vec);
@@ -491,7 +495,7 @@ SLLM_EXPORT int sllm_head_gate(void* x, int64_t ldx, const void* gate, int64_t l
 // part out (then r, positions and the tables are unused).
 SLLM_EXPORT int sllm_latent_small(const void* x, int64_t ldx, int64_t hsx, const void* w, void* out,
                                   int64_t ldo, int64_t hso, int n_tokens, int H, int K, int J,
-                                  const void* gate, int64_t ldg, int r, int tail,
+                                  const void* gate, int64_t ldg, int gate_wide, int r, int tail,
                                   const int* positions, const float* cos_t, const float* sin_t,
                                   int rot_dims, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
@@ -505,12 +509,12 @@ SLLM_EXPORT int sllm_latent_small(const void* x, int64_t ldx, int64_t hsx, const
     if (dtype == 0)
         return (int)sllm_launch_pdl(latent_small_kernel<float>, grid, dim3(256), smem, stream,
                                     (const float*)x, ldx, hsx, (const float*)w, (float*)out, ldo,
-                                    hso, n_tokens, K, J, (const float*)gate, ldg, r, tail,
+                                    hso, n_tokens, K, J, (const float*)gate, ldg, gate_wide, r, tail,
                                     positions, cos_t, sin_t, rot_dims);
     if (dtype == 1)
         return (int)sllm_launch_pdl(latent_small_kernel<bf16>, grid, dim3(256), smem, stream,
                                     (const bf16*)x, ldx, hsx, (const bf16*)w, (bf16*)out, ldo, hso,
-                                    n_tokens, K, J, (const bf16*)gate, ldg, r, tail, positions,
+                                    n_tokens, K, J, (const bf16*)gate, ldg, gate_wide, r, tail, positions,
                                     cos_t, sin_t, rot_dims);
     return (int)cudaErrorInvalidValue;
 }

@@ -43,7 +43,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z,
         for (int e = lane; e < n_total; e += 32) {
             const float s = 1.0f / (1.0f + expf(-z[e]));
             score[e] = s;
-            choice[e] = s + corr[e];
+            choice[e] = corr ? s + corr[e] : s;
         }
     } else {
         float m = -INFINITY;
@@ -59,7 +59,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z,
         for (int e = lane; e < n_total; e += 32) {
             const float s = score[e] / sum;
             score[e] = s;
-            choice[e] = s + corr[e];
+            choice[e] = corr ? s + corr[e] : s;
         }
     }
     __syncwarp();
@@ -152,8 +152,10 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z,
     }
 }
 
-// logits: float32 [N, n_total]; shared memory: warps * (2 n_total + 2 n_groups) floats.
-__global__ void moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ corr,
+// logits: float32 [N, n_total], rows ldl apart; corr may be null (no correction); shared
+// memory: warps * (2 n_total + 2 n_groups) floats.
+__global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ldl,
+                                 const float* __restrict__ corr,
                                  const int* __restrict__ token_row, int N, int n_total,
                                  int n_real, int n_groups, int keep, int top,
                                  int* __restrict__ ids, float* __restrict__ weights,
@@ -171,7 +173,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
         }
         return;
     }
-    route_token(logits + (int64_t)n * n_total, corr,
+    route_token(logits + (int64_t)n * ldl, corr,
                 smem + (size_t)warp * (2 * n_total + 2 * n_groups), n_total, n_real, n_groups, keep,
                 top, lane, ids + (int64_t)n * top, weights + (int64_t)n * top, counts, flags);
 }
@@ -183,7 +185,8 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
 // Shared memory: 8 warps' routing scratch, then counts [E], offsets [E + 1], cursor [E].
 constexpr int MOE_SMALL_WARPS = 8;
 __global__ void __launch_bounds__(MOE_SMALL_WARPS * 32)
-moe_route_small_kernel(const float* __restrict__ logits, const float* __restrict__ corr,
+moe_route_small_kernel(const float* __restrict__ logits, int64_t ldl,
+                       const float* __restrict__ corr,
                        const int* __restrict__ token_row, int N, int n_total, int n_real,
                        int n_groups, int keep, int top, int* __restrict__ ids,
                        float* __restrict__ weights, int* __restrict__ meta, int max_tiles,
@@ -210,7 +213,7 @@ moe_route_small_kernel(const float* __restrict__ logits, const float* __restrict
             }
             continue;
         }
-        route_token(logits + (int64_t)n * n_total, corr, smem + (size_t)warp * per_warp, n_total,
+        route_token(logits + (int64_t)n * ldl, corr, smem + (size_t)warp * per_warp, n_total,
                     n_real, n_groups, keep, top, lane, ids + (int64_t)n * top,
                     weights + (int64_t)n * top, counts, flags);
     }
@@ -386,16 +389,19 @@ moe_product_kernel(const TIn* __restrict__ X, int64_t ldx, const TIn* __restrict
 }
 
 // One block per token.  y: float32 [P, d]; x: the feed-forward's own input [N, d]; shared (may
-// be null): the shared expert's output [N, d].
+// be null): the shared expert's output [N, d]; sg (may be null): its gate's 32-bit logit per
+// token, rows ldsg apart (the output is multiplied by sigmoid(sg)).
 template <typename T>
 __global__ void moe_combine_kernel(const float* __restrict__ y, const T* __restrict__ x,
-                                   const T* __restrict__ shared, const int* __restrict__ ids,
+                                   const T* __restrict__ shared, const float* __restrict__ sg,
+                                   int64_t ldsg, const int* __restrict__ ids,
                                    const float* __restrict__ weights,
                                    const int* __restrict__ pair_place, int top, int n_real, int d,
                                    T* __restrict__ out) {
     pdl_wait();
     pdl_trigger();
     const int64_t n = blockIdx.x;
+    const float fs = sg ? 1.0f / (1.0f + expf(-sg[n * ldsg])) : 1.0f;
     for (int e = threadIdx.x; e < d; e += blockDim.x) {
         float acc = 0.f;
         for (int k = 0; k < top; ++k) {
@@ -406,7 +412,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const T* __restr
                                          : y[(int64_t)pair_place[n * top + k] * d + e];
             acc = fmaf(w, v, acc);
         }
-        if (shared != nullptr) acc += to_float(shared[n * d + e]);
+        if (shared != nullptr) acc = fmaf(fs, to_float(shared[n * d + e]), acc);
         out[n * d + e] = from_float<T>(acc);
     }
 }
@@ -440,13 +446,15 @@ template <> struct Quad<__nv_bfloat16> {
 
 template <typename T>
 __global__ void moe_combine_vec_kernel(const float* __restrict__ y, const T* __restrict__ x,
-                                       const T* __restrict__ shared, const int* __restrict__ ids,
+                                       const T* __restrict__ shared, const float* __restrict__ sg,
+                                       int64_t ldsg, const int* __restrict__ ids,
                                        const float* __restrict__ weights,
                                        const int* __restrict__ pair_place, int top, int n_real,
                                        int d, T* __restrict__ out) {
     pdl_wait();
     pdl_trigger();
     const int64_t n = blockIdx.x;
+    const float fs = sg ? 1.0f / (1.0f + expf(-sg[n * ldsg])) : 1.0f;
     for (int e = 4 * threadIdx.x; e < d; e += 4 * blockDim.x) {
         float acc[4] = {0.f, 0.f, 0.f, 0.f}, v[4];
         for (int k = 0; k < top; ++k) {
@@ -461,7 +469,7 @@ __global__ void moe_combine_vec_kernel(const float* __restrict__ y, const T* __r
         if (shared != nullptr) {
             Quad<T>::load(shared + n * d + e, v);
 #pragma unroll
-            for (int q = 0; q < 4; ++q) acc[q] += v[q];
+            for (int q = 0; q < 4; ++q) acc[q] = fmaf(fs, v[q], acc[q]);
         }
         Quad<T>::store(out + n * d + e, acc);
     }
@@ -475,14 +483,15 @@ SLLM_EXPORT int sllm_moe_tile_rows() { return MOE_TM; }
 
 // work: int32, zero-filled by the caller: counts [E], then offsets [E + 1], cursor [E],
 // meta [1 + 3 * max_tiles].
-SLLM_EXPORT int sllm_moe_route(const float* logits, const float* corr, const int* token_row,
+SLLM_EXPORT int sllm_moe_route(const float* logits, int64_t ldl, const float* corr,
+                               const int* token_row,
                                int n_tokens, int n_total, int n_real, int n_groups, int keep,
                                int top, int* ids, float* weights, int* work, int max_tiles,
                                int tile_rows, int* pair_token, int* pair_place, int flags,
                                cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (n_total <= 0 || n_real < 0 || n_real > n_total || top < 1 || top > MOE_MAX_TOP ||
-        top > n_total || n_groups < 1 || n_total % n_groups || keep < 1 || keep > n_groups ||
+    if (n_total <= 0 || ldl < n_total || n_real < 0 || n_real > n_total || top < 1 ||
+        top > MOE_MAX_TOP || top > n_total || n_groups < 1 || n_total % n_groups || keep < 1 || keep > n_groups ||
         n_total > 4096 || tile_rows < 1)
         return (int)cudaErrorInvalidValue;
     const int warps = 4;
@@ -493,7 +502,7 @@ SLLM_EXPORT int sllm_moe_route(const float* logits, const float* corr, const int
     cudaError_t err = sllm_launch_pdl(moe_route_kernel, dim3((n_tokens + warps - 1) / warps),
                                       dim3(32 * warps),
                                       (size_t)warps * (2 * n_total + 2 * n_groups) * sizeof(float),
-                                      stream, logits, corr, token_row, n_tokens, n_total, n_real,
+                                      stream, logits, ldl, corr, token_row, n_tokens, n_total, n_real,
                                       n_groups, keep, top, ids, weights, counts, flags);
     if (err != cudaSuccess) return (int)err;
     if (n_real == 0) return 0;
@@ -513,15 +522,16 @@ SLLM_EXPORT int sllm_moe_route_small_smem(int n_total, int n_real, int n_groups)
 
 // The router, the plan, the scatter and the copy of the rows in one launch, for steps of few
 // tokens.  meta: int32 [1 + 3 * max_tiles]; x / rows_out (bfloat16, may be null): see the kernel.
-SLLM_EXPORT int sllm_moe_route_small(const float* logits, const float* corr, const int* token_row,
+SLLM_EXPORT int sllm_moe_route_small(const float* logits, int64_t ldl, const float* corr,
+                                     const int* token_row,
                                      int n_tokens, int n_total, int n_real, int n_groups, int keep,
                                      int top, int* ids, float* weights, int* meta, int max_tiles,
                                      int tile_rows, int* pair_token, int* pair_place,
                                      const void* x, int64_t ldx, int K, void* rows_out, int flags,
                                      cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (n_total <= 0 || n_real < 0 || n_real > n_total || top < 1 || top > MOE_MAX_TOP ||
-        top > n_total || n_groups < 1 || n_total % n_groups || keep < 1 || keep > n_groups ||
+    if (n_total <= 0 || ldl < n_total || n_real < 0 || n_real > n_total || top < 1 ||
+        top > MOE_MAX_TOP || top > n_total || n_groups < 1 || n_total % n_groups || keep < 1 || keep > n_groups ||
         tile_rows < 1 || max_tiles < 1)
         return (int)cudaErrorInvalidValue;
     if (rows_out != nullptr &&
@@ -530,7 +540,7 @@ SLLM_EXPORT int sllm_moe_route_small(const float* logits, const float* corr, con
     const int smem = sllm_moe_route_small_smem(n_total, n_real, n_groups);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     return (int)sllm_launch_pdl(moe_route_small_kernel, dim3(1), dim3(MOE_SMALL_WARPS * 32),
-                                (size_t)smem, stream, logits, corr, token_row, n_tokens, n_total,
+                                (size_t)smem, stream, logits, ldl, corr, token_row, n_tokens, n_total,
                                 n_real, n_groups, keep, top, ids, weights, meta, max_tiles,
                                 tile_rows, pair_token, pair_place, (const __nv_bfloat16*)x, ldx, K,
                                 (__nv_bfloat16*)rows_out, flags);
@@ -577,7 +587,8 @@ SLLM_EXPORT int sllm_moe_product(const void* X, int64_t ldx, const void* W, void
     return (int)err;
 }
 
-SLLM_EXPORT int sllm_moe_combine(const float* y, const void* x, const void* shared, const int* ids,
+SLLM_EXPORT int sllm_moe_combine(const float* y, const void* x, const void* shared,
+                                 const float* sg, int64_t ldsg, const int* ids,
                                  const float* weights, const int* pair_place, int n_tokens,
                                  int top, int n_real, int d, void* out, int dtype,
                                  cudaStream_t stream) {
@@ -589,22 +600,24 @@ SLLM_EXPORT int sllm_moe_combine(const float* y, const void* x, const void* shar
         while (vt < 256 && vt * 4 < d) vt <<= 1;
         if (dtype == 0)
             return (int)sllm_launch_pdl(moe_combine_vec_kernel<float>, dim3(n_tokens), dim3(vt), 0,
-                                        stream, y, (const float*)x, (const float*)shared, ids,
+                                        stream, y, (const float*)x, (const float*)shared, sg,
+                                        ldsg, ids,
                                         weights, pair_place, top, n_real, d, (float*)out);
         if (dtype == 1)
             return (int)sllm_launch_pdl(moe_combine_vec_kernel<bf16>, dim3(n_tokens), dim3(vt), 0,
-                                        stream, y, (const bf16*)x, (const bf16*)shared, ids,
+                                        stream, y, (const bf16*)x, (const bf16*)shared, sg,
+                                        ldsg, ids,
                                         weights, pair_place, top, n_real, d, (bf16*)out);
         return (int)cudaErrorInvalidValue;
     }
     const int threads = d >= 256 ? 256 : 128;
     if (dtype == 0)
         return (int)sllm_launch_pdl(moe_combine_kernel<float>, dim3(n_tokens), dim3(threads), 0,
-                                    stream, y, (const float*)x, (const float*)shared, ids, weights,
+                                    stream, y, (const float*)x, (const float*)shared, sg, ldsg, ids, weights,
                                     pair_place, top, n_real, d, (float*)out);
     if (dtype == 1)
         return (int)sllm_launch_pdl(moe_combine_kernel<bf16>, dim3(n_tokens), dim3(threads), 0,
-                                    stream, y, (const bf16*)x, (const bf16*)shared, ids, weights,
+                                    stream, y, (const bf16*)x, (const bf16*)shared, sg, ldsg, ids, weights,
                                     pair_place, top, n_real, d, (bf16*)out);
     return (int)cudaErrorInvalidValue;
 }

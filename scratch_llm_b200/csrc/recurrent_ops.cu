@@ -1,13 +1,18 @@
 // What stands around a linear recurrence in a recurrent mixer: the short causal convolution
 // over time with its carried inputs, and the per-head norm and gate of the read-out.
 //
-//   conv:   y[t, c] = silu( sum_j taps[c, j] * x[t - (K - 1 - j), c] ),  j = 0 .. K-1
-//           (the last tap multiplies the current token; before a sequence's start x is 0).
+//   conv:   y[t, c] = silu( bias[c] + sum_j taps[c, j] * x[t - (K - 1 - j), c] ),  j = 0 .. K-1
+//           (the last tap multiplies the current token; before a sequence's start x is 0; the
+//           bias is optional).
 //           A request's last K - 1 inputs are carried in its state slot, state[slot, s, c] with
 //           s = K - 2 the most recent, so that a row may bring any number of tokens per step.
 //   update: the state after the row's tokens (a launch of its own: the convolution of a row's
 //           first tokens reads the old state while its last tokens would overwrite it).
-//   read-out: out[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * gain * silu(gate[t, h, :])
+//   read-out: out[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * gain * silu(gate[t, h, :]),
+//           optionally with o divided first by max(|den[t, h]|, floor[t, h]) + 1e-6; or, with the
+//           gate ahead of the norm, y = o * silu(gate), each of several equal parts of y over
+//           its own root mean square, times gain
+//   gates of a scan with one decay and one input weight per head (gated_scan.cu)
 //
 // T is the dtype of matrix-product operands (float / bfloat16); taps, gains and the read-out
 // o are 32-bit.  Tokens whose row is -1 are padding: their outputs are zero, nothing is carried.
@@ -17,11 +22,47 @@ namespace sllm {
 
 constexpr int CONV_MAX_TAPS = 16;
 
+// V consecutive values (4: 16 or 8 bytes at a time, suitably aligned; 1: one by one).
+template <int V> __device__ __forceinline__ void load_few(const float* p, float* v) {
+    if (V == 4) {
+        const float4 r = *reinterpret_cast<const float4*>(p);
+        v[0] = r.x; v[V - 3] = r.y; v[V - 2] = r.z; v[V - 1] = r.w;
+    } else {
+        v[0] = p[0];
+    }
+}
+template <int V> __device__ __forceinline__ void load_few(const __nv_bfloat16* p, float* v) {
+    if (V == 4) {
+        const uint2 r = *reinterpret_cast<const uint2*>(p);
+        const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&r);
+        v[0] = __low2float(h[0]); v[V - 3] = __high2float(h[0]);
+        v[V - 2] = __low2float(h[1]); v[V - 1] = __high2float(h[1]);
+    } else {
+        v[0] = __bfloat162float(p[0]);
+    }
+}
+template <int V> __device__ __forceinline__ void store_few(float* p, const float* v) {
+    if (V == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[V - 3], v[V - 2], v[V - 1]);
+    else p[0] = v[0];
+}
+template <int V> __device__ __forceinline__ void store_few(__nv_bfloat16* p, const float* v) {
+    if (V == 4) {
+        uint2 r;
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&r);
+        h[0] = __floats2bfloat162_rn(v[0], v[V - 3]);
+        h[1] = __floats2bfloat162_rn(v[V - 2], v[V - 1]);
+        *reinterpret_cast<uint2*>(p) = r;
+    } else {
+        p[0] = __float2bfloat16_rn(v[0]);
+    }
+}
+
 // x: [n_tokens, ldx], the convolved channels are its first C columns.  out: [n_tokens, C].
 template <typename T>
 __global__ void conv_silu_kernel(const T* __restrict__ x, int64_t ldx,
-                                 const float* __restrict__ taps, int K,
-                                 const T* __restrict__ state, const int* __restrict__ token_row,
+                                 const float* __restrict__ taps, const float* __restrict__ bias,
+                                 int K, const T* __restrict__ state,
+                                 const int* __restrict__ token_row,
                                  const int* __restrict__ row_start,
                                  const int* __restrict__ row_slot, T* __restrict__ out, int C,
                                  int64_t n_tokens) {
@@ -39,7 +80,7 @@ __global__ void conv_silu_kernel(const T* __restrict__ x, int64_t ldx,
         }
         const int i = (int)(n - row_start[r]);           // index of the token within its row
         const T* st = state + (int64_t)row_slot[r] * (K - 1) * C;
-        float acc = 0.f;
+        float acc = bias ? bias[c] : 0.f;
         for (int j = 0; j < K; ++j) {
             const int back = K - 1 - j;                  // how many tokens before this one
             float v;
@@ -56,7 +97,8 @@ __global__ void conv_silu_kernel(const T* __restrict__ x, int64_t ldx,
 // taps_t is the taps' transpose [K, C], so that a thread's 8 taps of one time step are 32
 // consecutive bytes and a warp's are consecutive too.
 __global__ void conv_silu_vec_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx,
-                                     const float* __restrict__ taps_t, int K,
+                                     const float* __restrict__ taps_t,
+                                     const float* __restrict__ bias, int K,
                                      const __nv_bfloat16* __restrict__ state,
                                      const int* __restrict__ token_row,
                                      const int* __restrict__ row_start,
@@ -78,7 +120,7 @@ __global__ void conv_silu_vec_kernel(const __nv_bfloat16* __restrict__ x, int64_
             const bf16* st = state + (int64_t)row_slot[r] * (K - 1) * C;
             float acc[8];
 #pragma unroll
-            for (int w = 0; w < 8; ++w) acc[w] = 0.f;
+            for (int w = 0; w < 8; ++w) acc[w] = bias ? bias[c + w] : 0.f;
             for (int j = 0; j < K; ++j) {
                 const int back = K - 1 - j;
                 const bf16* src = back <= i ? x + (n - back) * ldx + c : st + (int64_t)(i + j) * C + c;
@@ -121,22 +163,30 @@ __global__ void conv_state_update_kernel(const T* __restrict__ x, int64_t ldx, i
 
 // grid (tokens, ceil(H / 4)); one warp per (token, head).  o: [n_tokens, H * V] float;
 // gate: rows ldg apart; out: rows ldo apart (a column slice of a wider buffer, or H * V).  gain has V entries (every head the same) or,
-// with gain_per_head, H * V.  gate_act: 0 = silu(gate), 1 = sigmoid(gate).
+// with gain_per_head, H * V.  gate_act: 0 = silu(gate), 1 = sigmoid(gate).  den / floor (may be
+// null): [n_tokens, H]; a head's o is first divided by max(|den|, floor) + 1e-6.
+constexpr float DIVISOR_FLOOR = 1e-6f;
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ gate, int64_t ldg,
-                      const float* __restrict__ gain, float eps, T* __restrict__ out, int64_t ldo,
-                      int H, int V, int gain_per_head, int gate_act) {
+                      const float* __restrict__ gain, float eps, const float* __restrict__ den,
+                      const float* __restrict__ floor, T* __restrict__ out, int64_t ldo, int H,
+                      int V, int gain_per_head, int gate_act) {
     pdl_wait();
     pdl_trigger();
     const int64_t n = blockIdx.x;
     const int head = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (head >= H) return;
     const float* src = o + (n * H + head) * V;
+    float by = 1.f;
+    if (den) by = 1.0f / (fmaxf(fabsf(den[n * H + head]), floor[n * H + head]) + DIVISOR_FLOOR);
     float ss = 0.f;
-    for (int j = lane; j < V; j += 32) ss += src[j] * src[j];
+    for (int j = lane; j < V; j += 32) {
+        const float v = src[j] * by;
+        ss += v * v;
+    }
     ss = warp_sum(ss);
-    const float inv = 1.0f / sqrtf(ss / (float)V + eps);
+    const float inv = by / sqrtf(ss / (float)V + eps);
     const T* g = gate + n * ldg + (int64_t)head * V;
     const float* gn = gain + (gain_per_head ? (int64_t)head * V : 0);
     T* dst = out + n * ldo + (int64_t)head * V;
@@ -270,14 +320,150 @@ lowrank_expand_kernel(const float* __restrict__ pre, int64_t ldp, const ExpandJo
     }
 }
 
+// The gate ahead of the norm: y = o * silu(gate), then each of `parts` equal parts of y over its
+// own root mean square, times gain [W].  o: float [n_tokens, W]; one CTA per (token, part), a
+// part of P = W / parts elements waits in shared memory between the two passes.  V: elements per
+// access (4 where P and the rows allow 16-byte reads of o, else 1).
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+gate_part_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, int64_t ldg,
+                      const float* __restrict__ gain, float eps, T* __restrict__ out, int64_t ldo,
+                      int W, int P) {
+    pdl_wait();
+    pdl_trigger();
+    extern __shared__ __align__(16) float gp_row[];     // [P]
+    __shared__ float scratch[33];
+    const int64_t n = blockIdx.x;
+    const int at = blockIdx.y * P;
+    float ss = 0.f;
+    for (int i = threadIdx.x * V; i < P; i += blockDim.x * V) {
+        float v[V], z[V];
+        load_few<V>(o + n * W + at + i, v);
+        load_few<V>(gate + n * ldg + at + i, z);
+#pragma unroll
+        for (int k = 0; k < V; ++k) {
+            v[k] *= z[k] / (1.0f + expf(-z[k]));
+            ss = fmaf(v[k], v[k], ss);
+            gp_row[i + k] = v[k];
+        }
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)P + eps);
+    for (int i = threadIdx.x * V; i < P; i += blockDim.x * V) {
+        float v[V];
+#pragma unroll
+        for (int k = 0; k < V; ++k) v[k] = gp_row[i + k] * inv * gain[at + i + k];
+        store_few<V>(out + n * ldo + at + i, v);
+    }
+}
+
+// Gates of a scan with one decay and one input weight per head (gated_scan.cu), from 32-bit
+// projections.  A state-space layer: b = softplus(x + bias), log_a = -exp(A_log) * b; element
+// by element.  pre: rows ldp apart, the first H columns.
+__global__ void ssd_gates_kernel(const float* __restrict__ pre, int64_t ldp,
+                                 const float* __restrict__ bias, const float* __restrict__ A_log,
+                                 float* __restrict__ log_a, float* __restrict__ b, int n_tokens,
+                                 int H) {
+    pdl_wait();
+    pdl_trigger();
+    for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < (int64_t)n_tokens * H;
+         i += (int64_t)gridDim.x * blockDim.x) {
+        const int64_t n = i / H;
+        const int h = (int)(i - n * H);
+        const float x = pre[n * ldp + h] + bias[h];
+        const float step = x > 20.f ? x : log1pf(expf(x));
+        b[i] = step;
+        log_a[i] = -expf(A_log[h]) * step;
+    }
+}
+
+// A matrix memory with exponential gates: pre holds the input gates' sums in columns [0, H), the
+// forget gates' in [H, 2H).  i = cap tanh((x_i + b_i) / cap), f = log sigmoid(cap tanh((x_f +
+// b_f) / cap)); a running maximum m (one per slot and head, carried in `running`) keeps the state
+// in range: m_t = max(f + m_(t-1), i), log_a = f + m_(t-1) - m_t, b = exp(i - m_t), floor =
+// exp(-m_t).  (log_a and i - m_t are at most 0.)
+struct MemoryGates {
+    const float* pre; int64_t ldp; const float* bi; const float* bf; float cap;
+    float* running; const int* row_start; const int* row_slot;
+    float* log_a; float* b; float* floor; int H;
+};
+__device__ __forceinline__ void memory_gate_inputs(const MemoryGates& a, int64_t n, int h, float& i,
+                                                   float& f) {
+    i = a.cap * tanhf((a.pre[n * a.ldp + h] + a.bi[h]) / a.cap);
+    const float z = a.cap * tanhf((a.pre[n * a.ldp + a.H + h] + a.bf[h]) / a.cap);
+    f = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
+}
+// Rows of one token each (and rows without tokens): a thread per (row, head).
+__global__ void memory_gates_step_kernel(const MemoryGates a, int n_rows) {
+    pdl_wait();
+    pdl_trigger();
+    const int idx = blockIdx.x * blockDim.x + threadIdx.x;
+    if (idx >= n_rows * a.H) return;
+    const int r = idx / a.H, h = idx - r * a.H;
+    const int64_t n = a.row_start[r];
+    if (a.row_start[r + 1] <= n) return;
+    float i, f;
+    memory_gate_inputs(a, n, h, i, f);
+    float* m = a.running + (int64_t)a.row_slot[r] * a.H + h;
+    const float before = *m, now = fmaxf(f + before, i);
+    a.log_a[n * a.H + h] = f + before - now;
+    a.b[n * a.H + h] = expf(i - now);
+    a.floor[n * a.H + h] = expf(-now);
+    *m = now;
+}
+// Rows of any length: a CTA per (head, row), 256 tokens at a time.  The running maximum is a scan
+// over pairs (F, M): a token maps m to max(F + m, M) with (F, M) = (f, i), and two maps in a
+// row are (F1 + F2, max(M1 + F2, M2)).
+__global__ void __launch_bounds__(256) memory_gates_kernel(const MemoryGates a) {
+    pdl_wait();
+    pdl_trigger();
+    __shared__ float wF[8], wM[8];
+    const int h = blockIdx.x, r = blockIdx.y;
+    const int t0 = a.row_start[r], n_new = a.row_start[r + 1] - t0;
+    if (n_new <= 0) return;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    float* m = a.running + (int64_t)a.row_slot[r] * a.H + h;
+    float carried = *m;
+    for (int c0 = 0; c0 < n_new; c0 += 256) {
+        const int t = c0 + tid;
+        float i = -INFINITY, f = 0.f;          // (tokens beyond the row change nothing)
+        if (t < n_new) memory_gate_inputs(a, t0 + t, h, i, f);
+        float F = f, M = i;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float Fp = __shfl_up_sync(0xffffffffu, F, o), Mp = __shfl_up_sync(0xffffffffu, M, o);
+            if (lane >= o) {
+                M = fmaxf(Mp + F, M);
+                F += Fp;
+            }
+        }
+        __syncthreads();                       // the last round's sums are no longer read
+        if (lane == 31) { wF[warp] = F; wM[warp] = M; }
+        __syncthreads();
+        float start = carried;                 // m ahead of this warp's tokens
+        for (int w = 0; w < warp; ++w) start = fmaxf(wF[w] + start, wM[w]);
+        const float Fp = __shfl_up_sync(0xffffffffu, F, 1), Mp = __shfl_up_sync(0xffffffffu, M, 1);
+        const float before = lane == 0 ? start : fmaxf(Fp + start, Mp);
+        if (t < n_new) {
+            const float now = fmaxf(f + before, i);
+            const int64_t at = (int64_t)(t0 + t) * a.H + h;
+            a.log_a[at] = f + before - now;
+            a.b[at] = expf(i - now);
+            a.floor[at] = expf(-now);
+        }
+        for (int w = 0; w < 8; ++w) carried = fmaxf(wF[w] + carried, wM[w]);
+    }
+    if (tid == 0) *m = carried;
+}
+
 }  // namespace sllm
 
 using namespace sllm;
 
 // dtype: 0 = float32, 1 = bfloat16 (of x, state, out, gate).
-// taps_t (may be null): the transpose [K, C] of taps, which the kernel with 16-byte accesses reads.
+// bias (may be null): [C].  taps_t (may be null): the transpose [K, C] of taps, which the kernel with 16-byte accesses reads.
 SLLM_EXPORT int sllm_conv_silu(const void* x, int64_t ldx, const float* taps,
-                               const float* taps_t, int K,
+                               const float* taps_t, const float* bias, int K,
                                const void* state, const int* token_row, const int* row_start,
                                const int* row_slot, void* out, int C, int n_tokens, int dtype,
                                cudaStream_t stream) {
@@ -288,7 +474,7 @@ SLLM_EXPORT int sllm_conv_silu(const void* x, int64_t ldx, const float* taps,
         int64_t vblocks = ((int64_t)n_tokens * (C / 8) + 255) / 256;
         if (vblocks > 148 * 32) vblocks = 148 * 32;
         conv_silu_vec_kernel<<<(int)vblocks, 256, 0, stream>>>(
-            (const __nv_bfloat16*)x, ldx, taps_t, K, (const __nv_bfloat16*)state, token_row,
+            (const __nv_bfloat16*)x, ldx, taps_t, bias, K, (const __nv_bfloat16*)state, token_row,
             row_start, row_slot, (__nv_bfloat16*)out, C, n_tokens);
         SLLM_LAUNCH_CHECK();
         return 0;
@@ -297,11 +483,11 @@ SLLM_EXPORT int sllm_conv_silu(const void* x, int64_t ldx, const float* taps,
     if (blocks > 148 * 32) blocks = 148 * 32;
     if (dtype == 0)
         conv_silu_kernel<float><<<(int)blocks, 256, 0, stream>>>(
-            (const float*)x, ldx, taps, K, (const float*)state, token_row, row_start, row_slot,
+            (const float*)x, ldx, taps, bias, K, (const float*)state, token_row, row_start, row_slot,
             (float*)out, C, n_tokens);
     else if (dtype == 1)
         conv_silu_kernel<__nv_bfloat16><<<(int)blocks, 256, 0, stream>>>(
-            (const __nv_bfloat16*)x, ldx, taps, K, (const __nv_bfloat16*)state, token_row,
+            (const __nv_bfloat16*)x, ldx, taps, bias, K, (const __nv_bfloat16*)state, token_row,
             row_start, row_slot, (__nv_bfloat16*)out, C, n_tokens);
     else
         return (int)cudaErrorInvalidValue;
@@ -328,20 +514,21 @@ SLLM_EXPORT int sllm_conv_state_update(const void* x, int64_t ldx, int K, void* 
 }
 
 SLLM_EXPORT int sllm_head_norm_gate(const float* o, const void* gate, int64_t ldg,
-                                    const float* gain, float eps, void* out, int64_t ldo,
-                                    int n_tokens, int H, int V, int gain_per_head, int gate_act,
+                                    const float* gain, float eps, const float* den,
+                                    const float* floor, void* out, int64_t ldo, int n_tokens, int H, int V, int gain_per_head, int gate_act,
                                     int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (H <= 0 || V <= 0 || gate_act < 0 || gate_act > 1 || ldo < (int64_t)H * V)
+    if (H <= 0 || V <= 0 || gate_act < 0 || gate_act > 1 || ldo < (int64_t)H * V ||
+        (den == nullptr) != (floor == nullptr))
         return (int)cudaErrorInvalidValue;
     dim3 grid(n_tokens, (H + 3) / 4);
     if (dtype == 0)
         head_norm_gate_kernel<float><<<grid, 128, 0, stream>>>(o, (const float*)gate, ldg, gain,
-                                                               eps, (float*)out, ldo, H, V,
+                                                               eps, den, floor, (float*)out, ldo, H, V,
                                                                gain_per_head, gate_act);
     else if (dtype == 1)
         head_norm_gate_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>(
-            o, (const __nv_bfloat16*)gate, ldg, gain, eps, (__nv_bfloat16*)out, ldo, H, V,
+            o, (const __nv_bfloat16*)gate, ldg, gain, eps, den, floor, (__nv_bfloat16*)out, ldo, H, V,
             gain_per_head, gate_act);
     else
         return (int)cudaErrorInvalidValue;
@@ -396,4 +583,66 @@ SLLM_EXPORT int sllm_lowrank_expand(const float* pre, int64_t ldp, int n_jobs, c
         pre, ldp, j[0], j[1], blocks0, n_tokens);
     SLLM_LAUNCH_CHECK();
     return 0;
+}
+
+// out = parts of o * silu(gate) over their root mean squares, times gain.  o: float [n_tokens, W];
+// gate / out: rows ldg / ldo apart.
+SLLM_EXPORT int sllm_gate_part_norm(const float* o, const void* gate, int64_t ldg,
+                                    const float* gain, float eps, void* out, int64_t ldo,
+                                    int n_tokens, int W, int parts, int dtype,
+                                    cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (W <= 0 || parts < 1 || parts > 65535 || W % parts || ldg < W || ldo < W)
+        return (int)cudaErrorInvalidValue;
+    const int P = W / parts;
+    const size_t smem = (size_t)P * sizeof(float);
+    if (smem > 160 * 1024) return (int)cudaErrorInvalidValue;
+    const bool vec = P % 4 == 0 && ldg % 4 == 0 && ldo % 4 == 0 &&
+                     !(((uintptr_t)o | (uintptr_t)gate | (uintptr_t)out) & 15);
+    typedef __nv_bfloat16 bf16;
+#define SLLM_GPN(T, V)                                                                           \
+    do {                                                                                         \
+        if (smem > 48 * 1024) {                                                                  \
+            cudaError_t e = cudaFuncSetAttribute(gate_part_norm_kernel<T, V>,                    \
+                                                 cudaFuncAttributeMaxDynamicSharedMemorySize,    \
+                                                 (int)smem);                                     \
+            if (e != cudaSuccess) return (int)e;                                                 \
+        }                                                                                        \
+        return (int)sllm_launch_pdl(gate_part_norm_kernel<T, V>, dim3(n_tokens, parts),          \
+                                    dim3(256), smem, stream, o, (const T*)gate, ldg, gain, eps,  \
+                                    (T*)out, ldo, W, P);                                         \
+    } while (0)
+    if (dtype == 0 && vec) SLLM_GPN(float, 4);
+    if (dtype == 0) SLLM_GPN(float, 1);
+    if (dtype == 1 && vec) SLLM_GPN(bf16, 4);
+    if (dtype == 1) SLLM_GPN(bf16, 1);
+#undef SLLM_GPN
+    return (int)cudaErrorInvalidValue;
+}
+
+SLLM_EXPORT int sllm_ssd_gates(const float* pre, int64_t ldp, const float* bias,
+                               const float* A_log, float* log_a, float* b, int n_tokens, int H,
+                               cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (H <= 0 || ldp < H) return (int)cudaErrorInvalidValue;
+    int64_t blocks = ((int64_t)n_tokens * H + 255) / 256;
+    if (blocks > 148 * 16) blocks = 148 * 16;
+    return (int)sllm_launch_pdl(ssd_gates_kernel, dim3((int)blocks), dim3(256), 0, stream, pre, ldp,
+                                bias, A_log, log_a, b, n_tokens, H);
+}
+
+// running: float [slots, H], read and written at the rows' slots.  one_each: no row brings more
+// than one token.
+SLLM_EXPORT int sllm_memory_gates(const float* pre, int64_t ldp, const float* bi, const float* bf,
+                                  float cap, float* running, const int* row_start,
+                                  const int* row_slot, float* log_a, float* b, float* floor,
+                                  int n_rows, int H, int one_each, cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    if (H <= 0 || ldp < 2 * (int64_t)H || !(cap > 0.f) || n_rows > 65535)
+        return (int)cudaErrorInvalidValue;
+    MemoryGates a = {pre, ldp, bi, bf, cap, running, row_start, row_slot, log_a, b, floor, H};
+    if (one_each)
+        return (int)sllm_launch_pdl(memory_gates_step_kernel, dim3((n_rows * H + 127) / 128),
+                                    dim3(128), 0, stream, a, n_rows);
+    return (int)sllm_launch_pdl(memory_gates_kernel, dim3(H, n_rows), dim3(256), 0, stream, a);
 }

@@ -16,7 +16,8 @@ import torch
 from ..config.spec import ModelSpec, PartSpec
 from ..kernels import ops
 from ..parts import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, POSITION_ENCODINGS, SIDE_INPUTS,
-                     STREAM_JOINS, TOKEN_MIXES, BuildContext, CacheView, KVSpec, StateSpec, make)
+                     STREAM_JOINS, TOKEN_EMBEDDINGS, TOKEN_MIXES, BuildContext, CacheView, KVSpec,
+                     StateSpec, make)
 from ..parts.linear import Linear
 from ..parts.stream import Current, Normed, StreamSink
 from ..weights.loader import ParamSpec
@@ -125,13 +126,21 @@ class DecoderModel:
                 raise ValueError(f"norm {spec.embed_norm.kind!r} cannot norm the stream in place, "
                                  "which the norm after the embedding does")
             self._named_parts.append((spec.embed_norm_name, self.embed_norm))
+        # something the embedding adds to the tokens' own vectors, for designs that have it
+        self.token_embedding = None
+        if spec.token_embedding is not None:
+            self.token_embedding = make(TOKEN_EMBEDDINGS, "token embedding", spec.token_embedding)
+            self._named_parts.append((spec.token_embedding_name, self.token_embedding))
+            if spec.position_sinusoid_base > 0:
+                raise ValueError("a token embedding beside sinusoidal positions is not built")
         # what the first run starts with, for the embedding (if that block says, its norm's
         # factor is one number per token and its gain a vector `weight`)
         first = self.blocks[spec.order[0].layer] if spec.order else None
         entry = first.entry() if first is not None and hasattr(first, "entry") else None
         self._first_entry = entry if (entry is not None and getattr(entry[0], "deferrable", False)
                                       and hasattr(entry[1], "accepts_normed")
-                                      and spec.embed_norm is None) else None
+                                      and spec.embed_norm is None
+                                      and spec.token_embedding is None) else None
         # the last run may prepare the final norm for the output matrix in steps that want the
         # logits of every token in order (decode steps), where no rows are gathered in between
         last = self.blocks[spec.order[-1].layer] if spec.order else None
@@ -153,8 +162,9 @@ class DecoderModel:
         for part in self.joins:
             seen.setdefault(id(part), part)
         seen.setdefault(id(self.final_norm), self.final_norm)
-        if self.embed_norm is not None:
-            seen.setdefault(id(self.embed_norm), self.embed_norm)
+        for part in (self.embed_norm, self.token_embedding):
+            if part is not None:
+                seen.setdefault(id(part), part)
         return list(seen.values())
 
     # --------------------------------------------------------------------------- weights
@@ -205,7 +215,8 @@ class DecoderModel:
     # ----------------------------------------------------------------------------- cache
 
     def cache_specs(self) -> tuple[list[KVSpec | None], list[StateSpec | None]]:
-        """What each cache entry needs: the spec of the run that writes it."""
+        """What each cache entry needs: the spec of the run that writes it.  What the embedding
+        carries per request is one more entry after them, without keys and values."""
         n = self.spec.n_cache_entries
         ids = sorted({r.cache for r in self.spec.order})
         if ids != list(range(n)):
@@ -245,6 +256,9 @@ class DecoderModel:
                                  f"have another shape ({have} against {need})")
             if have.window is not None and (need.window is None or need.window > have.window):
                 kv[run.cache] = KVSpec(have.n_kv_heads, have.head_dim, need.window, have.planes)
+        if self.token_embedding is not None and self.token_embedding.state_spec() is not None:
+            kv.append(None)
+            st.append(self.token_embedding.state_spec())
         return kv, st
 
     def _states_of(self, cache, entry: int):
@@ -276,12 +290,20 @@ class DecoderModel:
 
     # --------------------------------------------------------------------------- forward
 
-    def _embed(self, batch, resid: torch.Tensor):
+    def _embed(self, batch, resid: torch.Tensor, cache):
         """The tokens' embeddings into the stream.  In steps of a few tokens the first run's
         norm is prepared for the product after it on the way (returned as what is pending),
         where that norm and that product can (scratch_llm_b200.parts.stream)."""
         s = self.spec
         n, d = batch.n_tokens, s.hidden_size
+        if self.token_embedding is not None:
+            if self._first_wants_current and self.embedding.dtype != torch.float32:
+                raise ValueError("a first block that reads the stream as it is needs an embedding "
+                                 "that leaves a copy of it")
+            stateful = self.token_embedding.state_spec() is not None
+            self.token_embedding.embed(batch, self.embedding, resid, s.embedding_multiplier,
+                                       cache.states[s.n_cache_entries] if stateful else None)
+            return None
         if s.position_sinusoid_base > 0 or self._first_wants_current:
             # the stream, and its copy in the compute dtype for a first block whose branches
             # read the stream as it is
@@ -311,7 +333,7 @@ class DecoderModel:
         s = self.spec
         resid = torch.empty((batch.n_tokens, s.hidden_size), dtype=torch.float32,
                             device=self.ctx.device)
-        pending = self._embed(batch, resid)
+        pending = self._embed(batch, resid, cache)
         if self.embed_norm is not None:
             if pending is not None:
                 raise ValueError("a norm after the embedding needs an embedding that leaves "

@@ -47,6 +47,8 @@ EXTRA_LIBRARIES: dict[str, tuple[tuple[str, ...], tuple[str, ...]]] = {
     "sllm_latent_attention": (("latent_attention.cu",), ()),
     "sllm_layer_norm": (("layer_norm.cu",), ()),
     "sllm_norm_rope_cache": (("norm_rope_cache.cu",), ()),
+    "sllm_gated_scan": (("gated_scan.cu",), ()),
+    "sllm_sum_norm": (("sum_norm.cu",), ()),
 }
 
 
@@ -1121,14 +1123,19 @@ def qk_norm_kv_write(x: torch.Tensor, positions: torch.Tensor, token_row: torch.
 
 def conv_silu(x: torch.Tensor, taps: torch.Tensor, state: torch.Tensor | None,
               token_row: torch.Tensor, row_start: torch.Tensor, row_slot: torch.Tensor,
-              out: torch.Tensor, taps_t: torch.Tensor | None = None) -> torch.Tensor:
+              out: torch.Tensor, taps_t: torch.Tensor | None = None,
+              bias: torch.Tensor | None = None) -> torch.Tensor:
     """Short causal convolution over time and silu on the first C columns of ``x`` [N, >= C]:
     ``taps`` float32 [C, K] (the last tap is the current token's), ``state`` [slots, K - 1, C]
     the inputs carried from earlier steps (None when K is 1), ``out`` [N, C].  ``taps_t``: the
     taps' transpose [K, C] (contiguous), which lets bfloat16 rows of whole 16 bytes take the
-    kernel with 16-byte accesses."""
+    kernel with 16-byte accesses.  ``bias`` (float32 [C]) is added before silu."""
     _need(x, None, "x", contiguous=False)
     _need(taps, torch.float32, "taps")
+    if bias is not None:
+        _need(bias, torch.float32, "bias")
+        if bias.numel() != taps.shape[0]:
+            raise KernelError("conv_silu: one bias per channel")
     _need(out, x.dtype, "out")
     for t, name in ((token_row, "token_row"), (row_start, "row_start"), (row_slot, "row_slot")):
         _need(t, torch.int32, name)
@@ -1146,7 +1153,7 @@ def conv_silu(x: torch.Tensor, taps: torch.Tensor, state: torch.Tensor | None,
         if taps_t.shape != (k, c):
             raise KernelError("taps_t must be the transpose of taps")
     _check(_core("sllm_recurrent_ops").sllm_conv_silu(
-        _ptr(x), c_int64(x.stride(0)), _ptr(taps), _ptr(taps_t), c_int(k),
+        _ptr(x), c_int64(x.stride(0)), _ptr(taps), _ptr(taps_t), _ptr(bias), c_int(k),
         _ptr(state if k > 1 else None),
         _ptr(token_row), _ptr(row_start), _ptr(row_slot), _ptr(out), c_int(c),
         c_int(x.shape[0]), c_int(_code(x.dtype)), _stream()), "conv_silu")
@@ -1173,13 +1180,21 @@ def conv_state_update(x: torch.Tensor, n_taps: int, state: torch.Tensor, row_sta
 
 
 def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, gain: torch.Tensor, eps: float,
-                   out: torch.Tensor, n_heads: int, gate_activation: str = "silu") -> torch.Tensor:
+                   out: torch.Tensor, n_heads: int, gate_activation: str = "silu",
+                   divisor: tuple[torch.Tensor, torch.Tensor] | None = None) -> torch.Tensor:
     """out[n, h, :] = o[n, h, :] / sqrt(mean(o[n, h, :]^2) + eps) * gain * act(gate[n, h, :]);
     ``o`` float32 [N, H * V], ``gate`` [N, H * V] (may be a column slice), ``gain`` float32 [V]
     (the same for every head) or [H * V]; ``gate_activation``: "silu" or "sigmoid".  ``out`` may
-    be a column slice of a wider buffer."""
+    be a column slice of a wider buffer.  ``divisor = (den, floor)``, float32 [N, H]: a head's
+    ``o`` is first divided by ``max(|den|, floor) + 1e-6``."""
     _need(o, torch.float32, "o")
     _need(gate, out.dtype, "gate", contiguous=False)
+    den, floor = divisor if divisor is not None else (None, None)
+    for t, name in ((den, "den"), (floor, "floor")):
+        if t is not None:
+            _need(t, torch.float32, name)
+            if t.shape != (o.shape[0], n_heads):
+                raise KernelError("head_norm_gate: the divisor has one entry per token and head")
     _need(gain, torch.float32, "gain")
     _need(out, None, "out", contiguous=False)
     n, hv = o.shape
@@ -1194,9 +1209,9 @@ def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, gain: torch.Tensor, eps:
     except KeyError:
         raise KernelError(f"unknown gate activation {gate_activation!r}") from None
     _check(_core("sllm_recurrent_ops").sllm_head_norm_gate(
-        _ptr(o), _ptr(gate), c_int64(gate.stride(0)), _ptr(gain), c_float(eps), _ptr(out),
-        c_int64(out.stride(0)), c_int(n), c_int(n_heads), c_int(v), c_int(int(per_head)), c_int(act),
-        c_int(_code(out.dtype)), _stream()), "head_norm_gate")
+        _ptr(o), _ptr(gate), c_int64(gate.stride(0)), _ptr(gain), c_float(eps), _ptr(den),
+        _ptr(floor), _ptr(out), c_int64(out.stride(0)), c_int(n), c_int(n_heads), c_int(v),
+        c_int(int(per_head)), c_int(act), c_int(_code(out.dtype)), _stream()), "head_norm_gate")
     return out
 
 
@@ -1382,12 +1397,12 @@ MOE_SIGMOID, MOE_GROUP_TOP2, MOE_RAW_WEIGHTS = 1, 2, 4
 MOE_PLAIN, MOE_GATED, MOE_SQRELU = 0, 1, 2
 
 
-def moe_route(logits: torch.Tensor, correction: torch.Tensor, token_row: torch.Tensor | None,
+def moe_route(logits: torch.Tensor, correction: torch.Tensor | None, token_row: torch.Tensor | None,
               n_real: int, n_groups: int, keep: int, top: int, tile_rows: int | None = None,
               gather_from: torch.Tensor | None = None, flags: int = 0):
-    """Route every token of ``logits`` (float32 [N, outputs]) and sort the (token, choice) pairs
-    by expert (csrc/moe.cu).  Returns ``(ids [N, top], weights [N, top], pair_token [N * top],
-    pair_place [N * top], meta, max_tiles, rows)``; ``meta`` is the tile list of the grouped
+    """Route every token of ``logits`` (float32 [N, outputs], may be a column slice) and sort the
+    (token, choice) pairs by expert (csrc/moe.cu).  Returns ``(ids [N, top], weights [N, top],
+    pair_token [N * top], pair_place [N * top], meta, max_tiles, rows)``; ``meta`` is the tile list of the grouped
     products, in tiles of ``tile_rows`` rows (default: what :func:`moe_product` takes).
     ``gather_from`` (bfloat16 [N, K], K % 8 == 0): the caller wants the tokens' rows in the
     sorted order; ``rows`` is that copy where the router made it on its way (steps of few tokens,
@@ -1395,11 +1410,14 @@ def moe_route(logits: torch.Tensor, correction: torch.Tensor, token_row: torch.T
     ``flags``: ``MOE_SIGMOID`` scores are ``sigmoid(z)`` instead of a softmax over the outputs;
     ``MOE_GROUP_TOP2`` a group's score is the sum of its two largest choice scores instead of its
     largest; ``MOE_RAW_WEIGHTS`` the weights are the chosen scores, not divided by their sum."""
-    _need(logits, torch.float32, "logits")
-    _need(correction, torch.float32, "correction")
+    _need(logits, torch.float32, "logits", contiguous=False)
     n, n_total = logits.shape
-    if correction.numel() != n_total:
-        raise KernelError("correction must have one entry per router output")
+    if logits.stride(1) != 1:
+        raise KernelError("moe_route: the logits of a token must be neighbours")
+    if correction is not None:
+        _need(correction, torch.float32, "correction")
+        if correction.numel() != n_total:
+            raise KernelError("correction must have one entry per router output")
     if token_row is not None:
         _need(token_row, torch.int32, "token_row")
     dev = logits.device
@@ -1422,7 +1440,8 @@ def moe_route(logits: torch.Tensor, correction: torch.Tensor, token_row: torch.T
                 raise KernelError("gather_from must be bfloat16 [N, K] with rows of whole 16 bytes")
             rows = torch.empty((n * top, gather_from.shape[1]), dtype=torch.bfloat16, device=dev)
         _check(lib.sllm_moe_route_small(
-            _ptr(logits), _ptr(correction), _ptr(token_row), c_int(n), c_int(n_total),
+            _ptr(logits), c_int64(logits.stride(0)), _ptr(correction), _ptr(token_row), c_int(n),
+            c_int(n_total),
             c_int(n_real), c_int(n_groups), c_int(keep), c_int(top), _ptr(ids), _ptr(weights),
             _ptr(meta), c_int(max_tiles), c_int(tile_rows), _ptr(pair_token), _ptr(pair_place),
             _ptr(gather_from), c_int64(gather_from.stride(0) if gather_from is not None else 0),
@@ -1435,7 +1454,8 @@ def moe_route(logits: torch.Tensor, correction: torch.Tensor, token_row: torch.T
     zeros = torch.zeros(n_scratch + n * top, dtype=torch.int32, device=dev)
     work, pair_token = zeros[:n_scratch], zeros[n_scratch:]
     _check(lib.sllm_moe_route(
-        _ptr(logits), _ptr(correction), _ptr(token_row), c_int(n), c_int(n_total), c_int(n_real),
+        _ptr(logits), c_int64(logits.stride(0)), _ptr(correction), _ptr(token_row), c_int(n),
+        c_int(n_total), c_int(n_real),
         c_int(n_groups), c_int(keep), c_int(top), _ptr(ids), _ptr(weights), _ptr(work),
         c_int(max_tiles), c_int(tile_rows), _ptr(pair_token), _ptr(pair_place), c_int(flags),
         _stream()), "moe_route")
@@ -1510,10 +1530,16 @@ def moe_tc_product(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, meta: to
 
 
 def moe_combine(y: torch.Tensor, x: torch.Tensor, shared: torch.Tensor | None, ids: torch.Tensor,
-                weights: torch.Tensor, pair_place: torch.Tensor, n_real: int, out: torch.Tensor
-                ) -> torch.Tensor:
+                weights: torch.Tensor, pair_place: torch.Tensor, n_real: int, out: torch.Tensor,
+                shared_gate: torch.Tensor | None = None) -> torch.Tensor:
     """out[token] = sum of weight * (the chosen expert's row of ``y``, or ``x[token]`` for an
-    identity expert) in the order of the choices, plus ``shared[token]``."""
+    identity expert) in the order of the choices, plus ``shared[token]``, which is multiplied by
+    ``sigmoid(shared_gate[token])`` first if that (float32 [N, 1], may be a column slice) is
+    given."""
+    if shared_gate is not None:
+        _need(shared_gate, torch.float32, "shared_gate", contiguous=False)
+        if shared is None or shared_gate.shape != (x.shape[0], 1):
+            raise KernelError("moe_combine: a shared expert's gate has one number per token")
     _need(y, torch.float32, "y")
     _need(x, None, "x")
     _need(out, x.dtype, "out")
@@ -1526,7 +1552,9 @@ def moe_combine(y: torch.Tensor, x: torch.Tensor, shared: torch.Tensor | None, i
     if out.shape != (n, d) or y.shape[1] != d or ids.shape[0] != n:
         raise KernelError("moe_combine shapes")
     _check(_core("sllm_moe").sllm_moe_combine(
-        _ptr(y), _ptr(x), _ptr(shared), _ptr(ids), _ptr(weights), _ptr(pair_place), c_int(n),
+        _ptr(y), _ptr(x), _ptr(shared), _ptr(shared_gate),
+        c_int64(shared_gate.stride(0) if shared_gate is not None else 0), _ptr(ids), _ptr(weights),
+        _ptr(pair_place), c_int(n),
         c_int(top), c_int(n_real), c_int(d), _ptr(out), c_int(_code(x.dtype)), _stream()),
         "moe_combine")
     return out
@@ -1665,21 +1693,25 @@ def lowrank_expand(pre: torch.Tensor, col0: int, w2t: torch.Tensor, out: torch.T
 # ------------------------------------------------------------------------ latent attention
 
 def latent_prep(a: torch.Tensor, q_rank: int, kv_col: int, kv_rank: int, rot_dim: int,
-                q_gain: torch.Tensor, kv_gain: torch.Tensor, eps: float, positions: torch.Tensor,
-                token_row: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, cq: torch.Tensor,
-                pages: torch.Tensor, block_table: torch.Tensor, page_size: int,
-                write: bool) -> torch.Tensor:
+                q_gain: torch.Tensor | None, kv_gain: torch.Tensor, eps: float,
+                positions: torch.Tensor, token_row: torch.Tensor, cos: torch.Tensor,
+                sin: torch.Tensor, cq: torch.Tensor | None, pages: torch.Tensor,
+                block_table: torch.Tensor, page_size: int, write: bool) -> torch.Tensor | None:
     """What a latent attention does with its down projections ``a`` [N, ...] (csrc/
     latent_attention.cu): ``cq`` [N, q_rank] gets the RMS-normed query latent (columns 0 ..
     q_rank of ``a``, times ``q_gain``); the page place of every token gets the RMS-normed
     key/value latent (columns kv_col .. kv_col + kv_rank, times ``kv_gain``), behind it the
     shared key part (the next ``rot_dim`` columns) with its first ``2 * cos.shape[1]`` entries
     rotated by the token's position (entry i pairs with entry i + half), then zeros up to the
-    pages' vector size.  ``pages``: [n_pages, 1, 1, page_size, Dp]."""
+    pages' vector size.  ``pages``: [n_pages, 1, 1, page_size, Dp].  ``q_rank`` 0 (queries
+    without a latent): ``q_gain`` and ``cq`` are None, only the cached vectors are made."""
     _need(a, None, "a", contiguous=False)
-    _need(cq, a.dtype, "cq")
+    if q_rank:
+        _need(cq, a.dtype, "cq")
+        _need(q_gain, torch.float32, "q_gain")
+        if cq.shape != (a.shape[0], q_rank) or q_gain.numel() != q_rank:
+            raise KernelError("latent_prep: the query latent's shapes")
     _need(pages, a.dtype, "pages")
-    _need(q_gain, torch.float32, "q_gain")
     _need(kv_gain, torch.float32, "kv_gain")
     _need(positions, torch.int32, "positions")
     _need(token_row, torch.int32, "token_row")
@@ -1689,7 +1721,7 @@ def latent_prep(a: torch.Tensor, q_rank: int, kv_col: int, kv_rank: int, rot_dim
     n = a.shape[0]
     rot_dims = 2 * cos.shape[1]
     if a.stride(1) != 1 or a.shape[1] < max(q_rank, kv_col + kv_rank + rot_dim) \
-            or cq.shape != (n, q_rank) or q_gain.numel() != q_rank or kv_gain.numel() != kv_rank \
+            or kv_gain.numel() != kv_rank \
             or sin.shape != cos.shape or rot_dims > rot_dim or block_table.stride(1) != 1:
         raise KernelError("latent_prep shapes")
     if pages.dim() != 5 or pages.shape[1:4] != (1, 1, page_size) \
@@ -1783,8 +1815,8 @@ def latent_small(x: torch.Tensor, x_head_stride: int, w: torch.Tensor, out: torc
     """A product per head for steps of few tokens, in one launch with what follows it:
     ``out[n, h * out_head_stride + j] = f * sum_k x[n, h * x_head_stride + k] * w[h, k, j]`` for
     ``w`` [H, K, J] (the output index last).  ``gate`` [N, H] (may be a column slice): ``f =
-    sigmoid(gate[n, h])``.  ``rot = (rot_dim, positions, cos, sin)``: the head's next ``rot_dim``
-    entries of ``x`` go behind the J outputs, the first ``2 * cos.shape[1]`` of them rotated by
+    sigmoid(gate[n, h])``; [N, H * J]: ``f = sigmoid(gate[n, h * J + j])``.  ``rot = (rot_dim,
+    positions, cos, sin)``: the head's next ``rot_dim`` entries of ``x`` go behind the J outputs, the first ``2 * cos.shape[1]`` of them rotated by
     the token's position (as :func:`latent_q_rot` does), zeros behind them up to
     ``out_head_stride``."""
     _need(x, None, "x", contiguous=False)
@@ -1804,8 +1836,9 @@ def latent_small(x: torch.Tensor, x_head_stride: int, w: torch.Tensor, out: torc
             raise KernelError("latent_small: the rotated part's shapes")
     if gate is not None:
         _need(gate, x.dtype, "gate", contiguous=False)
-        if gate.shape != (n, h) or gate.stride(1) != 1:
-            raise KernelError("latent_small: gate must be [tokens, heads]")
+        if gate.shape not in ((n, h), (n, h * j)) or gate.stride(1) != 1:
+            raise KernelError("latent_small: gate must be [tokens, heads] or [tokens, heads * "
+                              "outputs]")
     if x.stride(1) != 1 or out.stride(1) != 1 or out.shape[0] != n \
             or (h - 1) * x_head_stride + k + r > x.shape[1] \
             or (h - 1) * out_head_stride + j + tail > out.shape[1] \
@@ -1814,7 +1847,8 @@ def latent_small(x: torch.Tensor, x_head_stride: int, w: torch.Tensor, out: torc
     _check(_core("sllm_latent_attention").sllm_latent_small(
         _ptr(x), c_int64(x.stride(0)), c_int64(x_head_stride), _ptr(w), _ptr(out),
         c_int64(out.stride(0)), c_int64(out_head_stride), c_int(n), c_int(h), c_int(k), c_int(j),
-        _ptr(gate), c_int64(gate.stride(0) if gate is not None else 0), c_int(r), c_int(tail),
+        _ptr(gate), c_int64(gate.stride(0) if gate is not None else 0),
+        c_int(int(gate is not None and j > 1 and gate.shape[1] == h * j)), c_int(r), c_int(tail),
         _ptr(positions), _ptr(cos), _ptr(sin), c_int(rot_dims), c_int(_code(x.dtype)), _stream()),
         "latent_small")
     return out
@@ -1923,3 +1957,235 @@ def norm_rope_kv_write(x: torch.Tensor, positions: torch.Tensor, token_row: torc
         c_int(block_table.stride(0)), c_int(page_size), c_int(x.shape[0]), c_int(n_heads),
         c_int(n_kv_heads), c_int(head_dim), c_int(int(has_kv)), c_int(int(write)),
         c_int(_code(x.dtype)), _stream()), "norm_rope_kv_write")
+
+
+# --------------------------------------------------------------- norms of a sum of terms
+
+SUM_NORM_MAX_TERMS = 4
+
+
+def sum_norm(resid: torch.Tensor, terms: Sequence[tuple[torch.Tensor, float]], gain: torch.Tensor,
+             eps: float, out: torch.Tensor, gain_b: torch.Tensor | None = None,
+             out_b: torch.Tensor | None = None, routed=None,
+             out_rows: torch.Tensor | None = None) -> torch.Tensor:
+    """``x = resid + sum(coef * term) + routed`` in 32-bit, then ``out = x / sqrt(mean(x^2) +
+    eps) * gain`` and, from the same pass, ``out_b`` likewise with ``gain_b``
+    (csrc/sum_norm.cu).  ``routed`` (an object with the fields of
+    :class:`scratch_llm_b200.parts.stream.RoutedSum`): a routed feed-forward's output that is not
+    added up yet.  Without ``out_rows`` the stream is updated in place; with ``out_rows`` (int32)
+    only those tokens are normed, and the stream is not written."""
+    _need(resid, torch.float32, "resid")
+    _need(out, None, "out")
+    n, d = resid.shape
+    if len(terms) > SUM_NORM_MAX_TERMS:
+        raise KernelError(f"sum_norm takes up to {SUM_NORM_MAX_TERMS} terms")
+    for t, _ in terms:
+        _need(t, out.dtype, "term")
+        if t.shape != (n, d):
+            raise KernelError("sum_norm: a term must have the stream's shape")
+    n_out = n
+    if out_rows is not None:
+        _need(out_rows, torch.int32, "out_rows")
+        n_out = out_rows.numel()
+    if (gain_b is None) != (out_b is None):
+        raise KernelError("sum_norm: a second gain comes with a second output")
+    for w, o in ((gain, out), (gain_b, out_b)):
+        if w is not None:
+            _need(w, torch.float32, "gain")
+            _need(o, out.dtype, "out")
+            if w.numel() != d or o.shape != (n_out, d):
+                raise KernelError("sum_norm shapes")
+    y = ids = weights = place = shared = gate = None
+    top = 0
+    if routed is not None:
+        y, ids, weights, place = routed.y, routed.ids, routed.weights, routed.place
+        shared, gate, top = routed.shared, routed.gate, routed.ids.shape[1]
+        _need(y, torch.float32, "y")
+        _need(ids, torch.int32, "ids")
+        _need(weights, torch.float32, "weights")
+        _need(place, torch.int32, "place")
+        if y.shape[1] != d or ids.shape[0] != n or place.numel() != n * top:
+            raise KernelError("sum_norm: the routed sum's shapes")
+        if shared is not None:
+            _need(shared, out.dtype, "shared")
+            if shared.shape != (n, d):
+                raise KernelError("sum_norm: the shared expert's output has the stream's shape")
+        if gate is not None:
+            _need(gate, torch.float32, "gate", contiguous=False)
+            if shared is None or gate.shape != (n, 1):
+                raise KernelError("sum_norm: a shared expert's gate has one number per token")
+    ptrs = (c_void_p * SUM_NORM_MAX_TERMS)(*[t.data_ptr() for t, _ in terms])
+    coefs = (c_float * SUM_NORM_MAX_TERMS)(*[float(c) for _, c in terms])
+    _check(_core("sllm_sum_norm").sllm_sum_norm(
+        _ptr(resid), ptrs, coefs, c_int(len(terms)), _ptr(y), _ptr(ids), _ptr(weights),
+        _ptr(place), c_int(top), _ptr(shared), _ptr(gate),
+        c_int64(gate.stride(0) if gate is not None else 0), _ptr(gain), _ptr(gain_b),
+        c_float(eps), _ptr(out), _ptr(out_b), _ptr(out_rows), c_int(n_out), c_int(d),
+        c_int(_code(out.dtype)), _stream()), "sum_norm")
+    return out
+
+
+def embed_pair(ids: torch.Tensor, positions: torch.Tensor, token_row: torch.Tensor,
+               row_start: torch.Tensor, row_slot: torch.Tensor, table: torch.Tensor,
+               pairs: torch.Tensor, last: torch.Tensor, mul_prev: int, mul_cur: int,
+               out: torch.Tensor, pending: torch.Tensor | None = None,
+               scale: float = 1.0) -> torch.Tensor:
+    """:func:`embed` plus a vector for the pair (previous token, token): ``out[n] = table[id] *
+    scale + pairs[(previous * mul_prev + id * mul_cur) mod buckets]`` for ``pairs`` [buckets + 1,
+    d], whose last row is taken by a sequence's first token.  ``last`` (int32 [slots]) carries each
+    request's last token from step to step; it is read and written here."""
+    for t, name in ((ids, "ids"), (positions, "positions"), (token_row, "token_row"),
+                    (row_start, "row_start"), (row_slot, "row_slot"), (last, "last")):
+        _need(t, torch.int32, name)
+    if pending is not None:
+        _need(pending, torch.int32, "pending")
+    _need(table, None, "table")
+    _need(pairs, table.dtype, "pairs")
+    _need(out, torch.float32, "out")
+    n, d = ids.numel(), table.shape[1]
+    if out.shape != (n, d) or pairs.dim() != 2 or pairs.shape[1] != d or pairs.shape[0] < 2:
+        raise KernelError("embed_pair shapes")
+    _check(_core("sllm_sum_norm").sllm_embed_pair(
+        _ptr(ids), _ptr(pending), _ptr(positions), _ptr(token_row), _ptr(row_start),
+        _ptr(row_slot), _ptr(table), _ptr(pairs), _ptr(last), c_int64(mul_prev), c_int64(mul_cur),
+        c_int64(pairs.shape[0] - 1), c_float(scale), _ptr(out), c_int(n), c_int(d),
+        c_int(_code(table.dtype)), _stream()), "embed_pair")
+    return out
+
+
+# ------------------------------------------- recurrences with one decay and one weight per head
+
+#: the scan takes key sizes up to this
+GATED_SCAN_MAX_KEY_DIM = 1024
+#: rows of at least this many tokens take the chunk kernels where these take the sizes
+GATED_SCAN_MIN_CHUNKED = 32
+
+
+def gated_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: torch.Tensor,
+               weight: torch.Tensor, state: torch.Tensor, row_start: torch.Tensor,
+               row_slot: torch.Tensor, out: torch.Tensor, n_rows: int, n_groups: int, key_dim: int,
+               value_dim: int, longest: int, ones_out: torch.Tensor | None = None,
+               skip: torch.Tensor | None = None, scale: float = 1.0,
+               min_chunked: int | None = None) -> torch.Tensor:
+    """The recurrence ``S <- exp(log_decay) S + weight k v^T``, ``out = scale S^T q + skip v`` over
+    the packed batch (csrc/gated_scan.cu): ``q``, ``k`` [N, G * key_dim] and ``v`` [N, H *
+    value_dim] (may be column slices; head h reads group ``h // (H / G)``), ``log_decay`` (at
+    most 0) and ``weight`` float32 [N, H], ``skip`` float32 [H].  ``state`` float32 [slots, H,
+    value_dim, key_dim] is read and written at the rows' slots; with ``ones_out`` (float32 [N, H])
+    it is [slots, H, value_dim + 1, key_dim] and its last column belongs to a value that is
+    always 1 (a normaliser), whose read-out (times ``scale``) goes there.  ``longest``: the most
+    tokens a row brings (an upper bound).  ``min_chunked``: rows of at least so many tokens run in
+    chunks on the tensor cores (bfloat16, sizes in multiples of 16 and 8; 0: never)."""
+    _need(q, None, "q", contiguous=False)
+    _need(k, q.dtype, "k", contiguous=False)
+    _need(v, q.dtype, "v", contiguous=False)
+    for t, name in ((log_decay, "log_decay"), (weight, "weight"), (state, "state"), (out, "out")):
+        _need(t, torch.float32, name)
+    _need(row_start, torch.int32, "row_start")
+    _need(row_slot, torch.int32, "row_slot")
+    n, n_heads = log_decay.shape
+    ones = int(ones_out is not None)
+    for t, width in ((q, n_groups * key_dim), (k, n_groups * key_dim), (v, n_heads * value_dim)):
+        if t.shape != (n, width) or t.stride(1) != 1:
+            raise KernelError("gated_scan: q, k and v are [tokens, groups or heads * size]")
+    if n_heads % n_groups or weight.shape != (n, n_heads) or out.shape != (n, n_heads * value_dim) \
+            or state.shape[1:] != (n_heads, value_dim + ones, key_dim):
+        raise KernelError("gated_scan shapes")
+    if not 1 <= key_dim <= GATED_SCAN_MAX_KEY_DIM:
+        raise KernelError(f"gated_scan takes key sizes up to {GATED_SCAN_MAX_KEY_DIM}, got "
+                          f"{key_dim}")
+    if ones:
+        _need(ones_out, torch.float32, "ones_out")
+        if ones_out.shape != (n, n_heads):
+            raise KernelError("gated_scan: ones_out is [tokens, heads]")
+    if skip is not None:
+        _need(skip, torch.float32, "skip")
+        if skip.numel() != n_heads:
+            raise KernelError("gated_scan: one skip weight per head")
+    lib = _core("sllm_gated_scan")
+    if min_chunked is None:
+        min_chunked = GATED_SCAN_MIN_CHUNKED
+    aligned = all(t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in (q, k, v))
+    chunked = bool(min_chunked and longest >= min_chunked and q.dtype == torch.bfloat16 and aligned
+                   and lib.sllm_gated_scan_chunks_fit(c_int(key_dim), c_int(value_dim)))
+    dS = decay = None
+    if chunked:
+        slots = n // int(lib.sllm_gated_scan_chunk()) + n_rows + 1
+        dS = torch.empty((slots, n_heads, value_dim + ones, key_dim), dtype=torch.float32,
+                         device=q.device)
+        decay = torch.empty((slots, n_heads), dtype=torch.float32, device=q.device)
+    _check(lib.sllm_gated_scan(
+        _ptr(q), c_int64(q.stride(0)), _ptr(k), c_int64(k.stride(0)), _ptr(v),
+        c_int64(v.stride(0)), _ptr(log_decay), _ptr(weight), _ptr(state), _ptr(row_start),
+        _ptr(row_slot), _ptr(out), _ptr(ones_out), _ptr(skip), c_float(scale), c_int(n),
+        c_int(n_rows), c_int(n_heads), c_int(n_groups), c_int(key_dim), c_int(value_dim),
+        c_int(ones), c_int(int(chunked)), c_int(min_chunked), c_int(longest), _ptr(dS),
+        _ptr(decay), c_int(_code(q.dtype)), _stream()),
+        "gated_scan_chunked" if chunked else "gated_scan")
+    return out
+
+
+def ssd_gates(pre: torch.Tensor, bias: torch.Tensor, a_log: torch.Tensor,
+              log_decay: torch.Tensor, weight: torch.Tensor) -> None:
+    """A state-space layer's gates for :func:`gated_scan` (csrc/recurrent_ops.cu): ``weight =
+    softplus(pre + bias)``, ``log_decay = -exp(a_log) * weight``; all float32, ``pre`` [N, H] may
+    be a column slice."""
+    _need(pre, torch.float32, "pre", contiguous=False)
+    for t, name in ((bias, "bias"), (a_log, "a_log"), (log_decay, "log_decay"),
+                    (weight, "weight")):
+        _need(t, torch.float32, name)
+    n, h = pre.shape
+    if pre.stride(1) != 1 or bias.numel() != h or a_log.numel() != h \
+            or log_decay.shape != (n, h) or weight.shape != (n, h):
+        raise KernelError("ssd_gates shapes")
+    _check(_core("sllm_recurrent_ops").sllm_ssd_gates(
+        _ptr(pre), c_int64(pre.stride(0)), _ptr(bias), _ptr(a_log), _ptr(log_decay),
+        _ptr(weight), c_int(n), c_int(h), _stream()), "ssd_gates")
+
+
+def memory_gates(pre: torch.Tensor, bias_i: torch.Tensor, bias_f: torch.Tensor, cap: float,
+                 running: torch.Tensor, row_start: torch.Tensor, row_slot: torch.Tensor,
+                 n_rows: int, log_decay: torch.Tensor, weight: torch.Tensor,
+                 floor: torch.Tensor, one_each: bool = False) -> None:
+    """A matrix memory's exponential gates for :func:`gated_scan` (csrc/recurrent_ops.cu), kept
+    in range by a running maximum per head (``running`` float32 [slots, H], read and written at
+    the rows' slots): with ``i = cap tanh((pre_i + bias_i) / cap)`` and ``f = log sigmoid(cap
+    tanh((pre_f + bias_f) / cap))``, ``m <- max(f + m, i)``; ``log_decay = f + m_before - m``,
+    ``weight = exp(i - m)``, ``floor = exp(-m)``.  ``pre`` float32 [N, 2 H] (may be a column
+    slice): the input gates, then the forget gates.  ``one_each``: no row brings more than one
+    token."""
+    _need(pre, torch.float32, "pre", contiguous=False)
+    for t, name in ((bias_i, "bias_i"), (bias_f, "bias_f"), (running, "running"),
+                    (log_decay, "log_decay"), (weight, "weight"), (floor, "floor")):
+        _need(t, torch.float32, name)
+    _need(row_start, torch.int32, "row_start")
+    _need(row_slot, torch.int32, "row_slot")
+    n, h = log_decay.shape
+    if pre.stride(1) != 1 or pre.shape != (n, 2 * h) or bias_i.numel() != h \
+            or bias_f.numel() != h or weight.shape != (n, h) or floor.shape != (n, h) \
+            or running.shape[1:] != (h,):
+        raise KernelError("memory_gates shapes")
+    _check(_core("sllm_recurrent_ops").sllm_memory_gates(
+        _ptr(pre), c_int64(pre.stride(0)), _ptr(bias_i), _ptr(bias_f), c_float(cap),
+        _ptr(running), _ptr(row_start), _ptr(row_slot), _ptr(log_decay), _ptr(weight),
+        _ptr(floor), c_int(n_rows), c_int(h), c_int(int(one_each)), _stream()), "memory_gates")
+
+
+def gate_part_norm(o: torch.Tensor, gate: torch.Tensor, gain: torch.Tensor, eps: float,
+                   parts: int, out: torch.Tensor) -> torch.Tensor:
+    """``y = o * silu(gate)``, then each of ``parts`` equal parts of a token's ``y`` over its own
+    root mean square (eps inside the root), times ``gain``: the gate comes before the norm.
+    ``o`` float32 [N, W], ``gate`` [N, W] (may be a column slice), ``gain`` float32 [W]."""
+    _need(o, torch.float32, "o")
+    _need(gate, out.dtype, "gate", contiguous=False)
+    _need(gain, torch.float32, "gain")
+    _need(out, None, "out", contiguous=False)
+    n, w = o.shape
+    if gate.shape != (n, w) or out.shape != (n, w) or gate.stride(1) != 1 or out.stride(1) != 1 \
+            or gain.numel() != w or parts < 1 or w % parts:
+        raise KernelError("gate_part_norm shapes")
+    _check(_core("sllm_recurrent_ops").sllm_gate_part_norm(
+        _ptr(o), _ptr(gate), c_int64(gate.stride(0)), _ptr(gain), c_float(eps), _ptr(out),
+        c_int64(out.stride(0)), c_int(n), c_int(w), c_int(parts), c_int(_code(out.dtype)),
+        _stream()), "gate_part_norm")
+    return out

@@ -17,6 +17,8 @@ Mixer              ``forward(x, batch, cache, write, position) -> [N, hidden]``;
                    caches through ``kv_spec()`` (paged keys and values) and ``state_spec()``
                    (fixed-size state per request)
 FeedForward        ``forward(x) -> [N, hidden]``
+TokenEmbedding     ``embed(batch, table, resid, scale, state)``: the embedded tokens with something
+                   beside their own vectors, into the stream
 StreamJoin         ``forward(resid, first) -> resid``: the stream joined with the embedding
                    output, before a run that the model's run order marks
 Block              ``forward(resid, pending, batch, cache, write) -> pending``: the arrangement
@@ -174,6 +176,20 @@ class SideInput(Part):
     ids, positions or rows) beside the stream: ``forward(x, batch) -> [N, hidden]``."""
 
     def forward(self, x: torch.Tensor, batch: "StepBatch") -> torch.Tensor:
+        raise NotImplementedError
+
+
+class TokenEmbedding(Part):
+    """Something that the embedding adds to the tokens' own vectors (from their neighbours, for
+    instance): ``embed`` fills the 32-bit stream with ``table[token] * scale`` plus its own
+    contribution.  What it carries from token to token per live request it states in
+    ``state_spec()`` and receives as ``state``."""
+
+    def state_spec(self) -> "StateSpecs":
+        return None
+
+    def embed(self, batch: "StepBatch", table: torch.Tensor, resid: torch.Tensor, scale: float,
+              state) -> None:
         raise NotImplementedError
 
 

@@ -252,3 +252,43 @@ class SharedNormBlock(Block):
         if self.feed_forward is not None:
             out = out + Terms.of(self.feed_forward.forward(h), self.residual_mult)
         return out
+
+
+@register_block("parallel_norms")
+class ParallelNormsBlock(Block):
+    """Two branches side by side, each behind a norm of its own, both of the same stream:
+    ``x <- x + (Mixer(norm_a(x)) + FeedForward(norm_b(x)))`` (the feed-forward comes with its norm,
+    or both are left out).  One pass over the stream gives both norms (``forward_pair``), and it
+    takes in what the layer before left pending: the branches' outputs are handed on as a
+    weighted sum (:class:`~.stream.Terms`), the routed feed-forward's before it is added up
+    (:class:`~.stream.RoutedSum`) where the norm takes that."""
+
+    ROLES = {"mixer": "mixer", "mixer_norm": "norm", "feed_forward": "feed_forward",
+             "feed_forward_norm": "norm", "position": "position"}
+    OPTIONAL_ROLES = frozenset({"feed_forward", "feed_forward_norm"})
+    pad_safe = True   # the arrangement itself touches no token: its parts decide
+
+    def __init__(self, mixer: Mixer, mixer_norm: Norm, position: PositionEncoding,
+                 feed_forward: FeedForward | None = None,
+                 feed_forward_norm: Norm | None = None) -> None:
+        if (feed_forward is None) != (feed_forward_norm is None):
+            raise ValueError("a feed-forward and the norm in front of it come together")
+        if not getattr(mixer_norm, "takes_terms", False):
+            raise ValueError("a parallel_norms block needs norms that take a sum of terms as what "
+                             "is pending (takes_terms)")
+        if feed_forward_norm is not None and not (hasattr(mixer_norm, "pairs_with")
+                                                  and mixer_norm.pairs_with(feed_forward_norm)):
+            raise ValueError("the two norms of a parallel_norms block must pair up (pairs_with)")
+        self.mixer, self.mixer_norm, self.position = mixer, mixer_norm, position
+        self.feed_forward, self.feed_forward_norm = feed_forward, feed_forward_norm
+        self._lazy = getattr(feed_forward, "hands_on_routed", False) and \
+            getattr(mixer_norm, "takes_routed", False)
+
+    def forward(self, resid: torch.Tensor, pending, batch, cache: CacheView, write: bool):
+        if self.feed_forward is None:
+            h = self.mixer_norm.forward(resid, pending)
+            return Terms.of(self.mixer.forward(h, batch, cache, write, self.position))
+        h, g = self.mixer_norm.forward_pair(resid, pending, self.feed_forward_norm)
+        a = Terms.of(self.mixer.forward(h, batch, cache, write, self.position))
+        f = self.feed_forward.forward(g, lazy=True) if self._lazy else self.feed_forward.forward(g)
+        return a + Terms.of(f)

@@ -22,6 +22,13 @@ the layer's rotary position encoding, whose tables have ``rot_dims / 2`` columns
 Every size is a constructor argument; ``gate`` False leaves the output gate out.  Norms,
 rotation, scores and softmax are 32-bit; the cache and the products' operands have the compute
 dtype.
+
+Options for other designs: ``q_rank`` None (queries without a latent, ``q = W_q x``, tensor ``q``
+instead of ``dq``, ``dq.norm`` and ``uq``; all of the mixer's products of x are then one),
+``gate="wide"`` (a gate per channel, ``g`` [H * value_dim, hidden]) and ``adjacent_pairs=n`` (of
+the first n entries of the rotated part, entry 2i turns with entry 2i + 1: the rows of the
+queries' and of the shared key's rotated parts are put into the split-half order once at load,
+which changes no score).
 """
 
 from __future__ import annotations
@@ -49,10 +56,19 @@ class LatentAttention(Mixer):
     pad_safe = True   # padding tokens are not stored; rows without tokens leave the kernels
 
     def __init__(self, hidden_size: int, n_heads: int, dim: int, rot_dim: int, value_dim: int,
-                 q_rank: int, kv_rank: int, scale: float, eps: float, gate: bool = True,
-                 names: Mapping[str, str] | None = None) -> None:
-        if min(hidden_size, n_heads, dim, value_dim, q_rank, kv_rank) < 1 or rot_dim < 0:
+                 q_rank: int | None, kv_rank: int, scale: float, eps: float,
+                 gate: bool | str = True, names: Mapping[str, str] | None = None,
+                 adjacent_pairs: int = 0) -> None:
+        if min(hidden_size, n_heads, dim, value_dim, kv_rank) < 1 or rot_dim < 0 \
+                or (q_rank is not None and q_rank < 1):
             raise ValueError("latent attention: sizes must be positive")
+        if gate not in (True, False, "wide"):
+            raise ValueError(f"gate must be True, False or 'wide', got {gate!r}")
+        self.gate_width = 0 if not gate else n_heads * value_dim if gate == "wide" else n_heads
+        if adjacent_pairs % 2 or not 0 <= adjacent_pairs <= rot_dim:
+            raise ValueError(f"adjacent_pairs must be even and at most {rot_dim}, got "
+                             f"{adjacent_pairs}")
+        self.adjacent_pairs = adjacent_pairs
         self.hidden_size, self.n_heads, self.dim, self.rot_dim = hidden_size, n_heads, dim, rot_dim
         self.value_dim, self.q_rank, self.kv_rank = value_dim, q_rank, kv_rank
         self.scale, self.eps, self.has_gate = float(scale), float(eps), bool(gate)
@@ -62,9 +78,9 @@ class LatentAttention(Mixer):
             raise ValueError(f"kv_rank + rot_dim = {kv_rank + rot_dim}: the attention kernels "
                              f"take cached vectors of up to {ops.SIMT_MAX_HEAD_DIM} entries")
         self.names = {"dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "dkv": "dkv",
-                      "dkv_norm": "dkv.norm", "uk": "uk", "uv": "uv", "g": "g", "o": "o",
+                      "q": "q", "dkv_norm": "dkv.norm", "uk": "uk", "uv": "uv", "g": "g", "o": "o",
                       **(names or {})}
-        self.down: Linear | None = None     # [dq; dkv; g] in one product
+        self.down: Linear | None = None     # [dq or q; dkv; g] in one product
         self.uq: Linear | None = None
         self.o: Linear | None = None
         self.uk = self.uk_t = self.uv = self.uv_t = self.q_gain = self.kv_gain = None
@@ -77,7 +93,7 @@ class LatentAttention(Mixer):
         return dtype == torch.bfloat16 and self.head_dim <= ops.MMA_MAX_HEAD_DIM
 
     def kernel_jobs(self, dtype: torch.dtype):
-        jobs = [ops.core_job("sllm_latent_attention")]
+        jobs = [ops.core_job("sllm_latent_attention"), ops.core_job("sllm_stream_ops")]
         if self._tensor_cores(dtype):
             jobs.append(ops.attention_mma_library(self.head_dim))
             if ops.attention_tc_supports(self.n_heads, 1, self.head_dim, 16, None):
@@ -88,27 +104,55 @@ class LatentAttention(Mixer):
 
     def param_specs(self) -> dict[str, ParamSpec]:
         n, H, d = self.names, self.n_heads, self.hidden_size
-        specs = {n["dq"]: ParamSpec((self.q_rank, d)),
-                 n["dq_norm"]: ParamSpec((self.q_rank,), "gain"),
-                 n["uq"]: ParamSpec((H * (self.dim + self.rot_dim), self.q_rank)),
-                 n["dkv"]: ParamSpec((self.kv_rank + self.rot_dim, d)),
+        wide = H * (self.dim + self.rot_dim)
+        specs = {n["dkv"]: ParamSpec((self.kv_rank + self.rot_dim, d)),
                  n["dkv_norm"]: ParamSpec((self.kv_rank,), "gain"),
                  n["uk"]: ParamSpec((H * self.dim, self.kv_rank)),
                  n["uv"]: ParamSpec((H * self.value_dim, self.kv_rank)),
                  n["o"]: ParamSpec((d, H * self.value_dim))}
+        if self.q_rank is None:
+            specs[n["q"]] = ParamSpec((wide, d))
+        else:
+            specs.update({n["dq"]: ParamSpec((self.q_rank, d)),
+                          n["dq_norm"]: ParamSpec((self.q_rank,), "gain"),
+                          n["uq"]: ParamSpec((wide, self.q_rank))})
         if self.has_gate:
-            specs[n["g"]] = ParamSpec((H, d))
+            specs[n["g"]] = ParamSpec((self.gate_width, d))
         return specs
+
+    def _split_half(self, rows: torch.Tensor) -> torch.Tensor:
+        """``rows`` [..., rot_dim, in] of a rotated part whose first n entries turn in pairs
+        (2i, 2i + 1), in the order that pairs i with i + n / 2."""
+        n = self.adjacent_pairs
+        order = [*range(0, n, 2), *range(1, n, 2), *range(n, self.rot_dim)]
+        return rows[..., order, :] if n else rows
 
     def load(self, tensors: Mapping[str, torch.Tensor], ctx: BuildContext) -> None:
         put = lambda t: t.to(device=ctx.device, dtype=ctx.dtype)  # noqa: E731
         f32 = lambda t: t.to(device=ctx.device, dtype=torch.float32).contiguous()  # noqa: E731
-        n, H = self.names, self.n_heads
-        blocks = [put(tensors[n["dq"]]), put(tensors[n["dkv"]])]
+        n, H, R = self.names, self.n_heads, self.kv_rank
+
+        def with_rotated(t: torch.Tensor, plain: int, heads: int) -> torch.Tensor:
+            t = put(t).view(heads, plain + self.rot_dim, t.shape[1])
+            return torch.cat([t[:, :plain], self._split_half(t[:, plain:])], 1).flatten(0, 1)
+
+        wide = tensors[n["q" if self.q_rank is None else "uq"]]
+        wide = with_rotated(wide, self.dim, H)
+        blocks = [wide if self.q_rank is None else put(tensors[n["dq"]]),
+                  with_rotated(tensors[n["dkv"]], R, 1)]
+        self.kv_col = blocks[0].shape[0]
+        self.gate_col = self.kv_col + blocks[1].shape[0]
         if self.has_gate:
+            if self.gate_width > H:     # a gate per channel: its columns start on 16 bytes
+                pad = -self.gate_col % 8
+                blocks.append(wide.new_zeros((pad, self.hidden_size)))
+                self.gate_col += pad
             blocks.append(put(tensors[n["g"]]))
+        if self.q_rank is None:         # whole rows of 16 bytes
+            total = sum(b.shape[0] for b in blocks)
+            blocks.append(wide.new_zeros((-total % 8, self.hidden_size)))
         self.down = Linear(torch.cat(blocks, 0).contiguous())
-        self.uq = Linear(put(tensors[n["uq"]]).contiguous())
+        self.uq = None if self.q_rank is None else Linear(wide.contiguous())
         self.o = Linear(put(tensors[n["o"]]).contiguous())
         self.uk = put(tensors[n["uk"]]).view(H, self.dim, self.kv_rank).contiguous()
         # [H, kv_rank, dim]: the absorb product's matrix with the reduction index last
@@ -120,7 +164,8 @@ class LatentAttention(Mixer):
         self._small = ctx.dtype == torch.bfloat16 \
             and ops.latent_small_supports(self.dim, self.kv_rank) \
             and ops.latent_small_supports(self.kv_rank, self.value_dim)
-        self.q_gain, self.kv_gain = f32(tensors[n["dq_norm"]]), f32(tensors[n["dkv_norm"]])
+        self.q_gain = None if self.q_rank is None else f32(tensors[n["dq_norm"]])
+        self.kv_gain = f32(tensors[n["dkv_norm"]])
 
     # ------------------------------------------------------------------------- forward
 
@@ -128,18 +173,22 @@ class LatentAttention(Mixer):
         if not getattr(position, "rotary_tables", False):
             raise ValueError("latent attention needs a rotary position encoding's tables")
         cos, sin = position.cos, position.sin
+        if self.adjacent_pairs and 2 * cos.shape[1] != self.adjacent_pairs:
+            raise ValueError("latent attention: the position encoding turns another number of "
+                             "entries than were put in order")
         H, d, r, R, V, Dp = (self.n_heads, self.dim, self.rot_dim, self.kv_rank, self.value_dim,
                              self.head_dim)
         n = x.shape[0]
-        a = self.down(x)                                        # [N, q_rank + R + r (+ H)]
-        cq = torch.empty((n, self.q_rank), dtype=a.dtype, device=a.device)
-        ops.latent_prep(a, self.q_rank, self.q_rank, R, r, self.q_gain, self.kv_gain, self.eps,
-                        batch.positions, batch.token_row, cos, sin, cq, cache.pages,
+        a = self.down(x)                                        # [N, (dq or q) + R + r (+ gate)]
+        cq = None if self.q_rank is None else torch.empty((n, self.q_rank), dtype=a.dtype,
+                                                          device=a.device)
+        ops.latent_prep(a, self.q_rank or 0, self.kv_col, R, r, self.q_gain, self.kv_gain,
+                        self.eps, batch.positions, batch.token_row, cos, sin, cq, cache.pages,
                         cache.block_table, cache.page_size, write)
-        q = self.uq(cq)                                         # [N, H * (d + r)]
+        q = a[:, :H * (d + r)] if self.q_rank is None else self.uq(cq)     # [N, H * (d + r)]
         qlat = torch.empty((n, H * Dp), dtype=q.dtype, device=q.device)
         small = self._small and n <= ops.LATENT_SMALL_MAX_TOKENS
-        gate = a[:, self.q_rank + R + r:] if self.has_gate else None
+        gate = a[:, self.gate_col:self.gate_col + self.gate_width] if self.has_gate else None
         if small:
             # steps of few tokens: absorb product and rotation in one launch, value product and
             # gate in another
@@ -152,7 +201,7 @@ class LatentAttention(Mixer):
             return self.o(o)
         if q.dtype == torch.bfloat16:
             # the library's batched product, one batch per head, straight into its columns
-            torch.bmm(q.view(n, H, d + r)[:, :, :d].transpose(0, 1), self.uk,
+            torch.bmm(q.unflatten(1, (H, d + r))[:, :, :d].transpose(0, 1), self.uk,
                       out=qlat.view(n, H, Dp)[:, :, :R].transpose(0, 1))
         else:
             ops.head_product(q, d + r, self.uk_t, qlat, Dp)
@@ -167,7 +216,9 @@ class LatentAttention(Mixer):
                       out=o.view(n, H, V).transpose(0, 1))
         else:
             ops.head_product(olat, Dp, self.uv, o, V)
-        if self.has_gate:
+        if self.gate_width > H:
+            ops.sigmoid_gate(o, gate)
+        elif self.has_gate:
             ops.head_gate(o, gate, H)
         return self.o(o)
 

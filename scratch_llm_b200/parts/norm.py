@@ -24,6 +24,8 @@ class RMSNorm(Norm):
     #: the norm's factor is one number per token: the product before it may prepare it and the
     #: product after it may apply it (scratch_llm_b200.parts.stream)
     deferrable = True
+    takes_terms = True    # forward() accepts a Terms as what is pending
+    takes_routed = True   # ... and a routed feed-forward's output in it
 
     def __init__(self, size: int, eps: float, name: str = "weight", offset: float = 0.0) -> None:
         """``name``: the gain's tensor name below the part's prefix; "" if the prefix itself is
@@ -54,7 +56,25 @@ class RMSNorm(Norm):
             delta = None
         n = resid.shape[0] if out_rows is None else out_rows.numel()
         out = torch.empty((n, self.size), dtype=self.dtype, device=resid.device)
+        if isinstance(delta, Terms):
+            return ops.sum_norm(resid, delta.items, self.weight, self.eps, out,
+                                routed=delta.routed, out_rows=out_rows)
         return ops.add_rmsnorm(resid, delta, self.weight, self.eps, out, out_rows)
+
+    def forward_pair(self, resid: torch.Tensor, delta, other: "RMSNorm"):
+        """``(self(x), other(x))`` of the same stream from one pass, for layers whose branches run
+        side by side behind a norm each (``pairs_with``)."""
+        if isinstance(delta, Current):
+            delta = None
+        terms = Terms(()) if delta is None else Terms.of(delta)
+        out = torch.empty((resid.shape[0], self.size), dtype=self.dtype, device=resid.device)
+        out_b = torch.empty_like(out)
+        ops.sum_norm(resid, terms.items, self.weight, self.eps, out, other.weight, out_b,
+                     routed=terms.routed)
+        return out, out_b
+
+    def pairs_with(self, other) -> bool:
+        return isinstance(other, RMSNorm) and (other.size, other.eps) == (self.size, self.eps)
 
     def add_normed(self, resid: torch.Tensor, delta: torch.Tensor,
                    cast_out: torch.Tensor | None = None, then: "RMSNorm | None" = None):

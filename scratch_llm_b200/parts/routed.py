@@ -18,7 +18,14 @@ Variants for other designs, each a constructor argument: ``score="sigmoid"`` (s 
 output by itself, instead of the softmax), ``group_score="top2"`` (a group's score is the sum of
 its two largest choice scores instead of its largest), ``renormalize=False`` (the weights are the
 chosen scores s themselves) and ``expert="sqrelu"`` (experts without a gate,
-``W_down(relu(W_up x)^2)``, tensors ``e<i>.{up,down}``).
+``W_down(relu(W_up x)^2)``, tensors ``e<i>.{up,down}``); ``correction=False`` (the choice is by the
+scores alone, there is no such tensor) and ``shared_gate=True`` (the shared expert's output is
+multiplied by ``sigmoid(w_sg . x)``, one number per token, tensor ``shared.sg``; its logit comes
+out of the router's product).  A softmax over all outputs whose chosen scores are divided by
+their sum is the softmax over the chosen outputs' logits alone.
+
+A block and a norm that take it get the output before it is added up (``lazy=True``:
+:class:`~.stream.RoutedSum`).
 
 Nothing of a step is read on the host: the router's kernel sorts the (token, choice) pairs by
 expert on the device and the grouped products walk a tile list, so steps can be recorded into
@@ -38,6 +45,7 @@ from .base import BuildContext, FeedForward
 from .feed_forward import SwiGLU
 from .linear import Linear
 from .registry import register_feed_forward
+from .stream import RoutedSum
 
 
 @register_feed_forward("routed_experts")
@@ -48,7 +56,8 @@ class RoutedExperts(FeedForward):
                  identity: int = 0, groups: int = 1, keep_groups: int = 1,
                  shared_size: int | None = None, score: str = "softmax",
                  group_score: str = "max", renormalize: bool = True,
-                 expert: str = "gated_silu") -> None:
+                 expert: str = "gated_silu", correction: bool = True,
+                 shared_gate: bool = False) -> None:
         total = experts + identity
         if experts < 0 or identity < 0 or total < 1:
             raise ValueError("a router needs at least one output")
@@ -71,6 +80,11 @@ class RoutedExperts(FeedForward):
         self.hidden_size, self.expert_size = hidden_size, expert_size
         self.experts, self.identity, self.top = experts, identity, top
         self.groups, self.keep_groups = groups, keep_groups
+        if shared_gate and shared_size is None:
+            raise ValueError("a shared expert's gate needs a shared expert")
+        self.has_correction, self.shared_gate = bool(correction), bool(shared_gate)
+        #: forward() takes lazy=: the output may be handed on before it is added up
+        self.hands_on_routed = identity == 0 and experts > 0
         self.shared = None if shared_size is None else SwiGLU(
             hidden_size, shared_size, names={"gate": "shared.gate", "up": "shared.up",
                                              "down": "shared.down"})
@@ -91,7 +105,11 @@ class RoutedExperts(FeedForward):
 
     def param_specs(self) -> dict[str, ParamSpec]:
         d, f, total = self.hidden_size, self.expert_size, self.experts + self.identity
-        specs = {"router": ParamSpec((total, d)), "correction": ParamSpec((total,), "gain")}
+        specs = {"router": ParamSpec((total, d))}
+        if self.has_correction:
+            specs["correction"] = ParamSpec((total,), "gain")
+        if self.shared_gate:
+            specs["shared.sg"] = ParamSpec((1, d))
         for e in range(self.experts):
             if self.first == ops.MOE_GATED:
                 specs[f"e{e}.gate"] = ParamSpec((f, d))
@@ -103,9 +121,13 @@ class RoutedExperts(FeedForward):
 
     def load(self, tensors: Mapping[str, torch.Tensor], ctx: BuildContext) -> None:
         put = lambda t: t.to(device=ctx.device, dtype=ctx.dtype)  # noqa: E731
-        self.router = Linear(put(tensors["router"]).contiguous())
-        self.correction = tensors["correction"].to(device=ctx.device,
-                                                   dtype=torch.float32).contiguous()
+        router = [put(tensors["router"])]
+        if self.shared_gate:      # one more output of the router's product
+            router.append(put(tensors["shared.sg"]))
+        self.router = Linear(torch.cat(router, 0).contiguous())
+        if self.has_correction:
+            self.correction = tensors["correction"].to(device=ctx.device,
+                                                       dtype=torch.float32).contiguous()
         if self.experts:
             # [E, 2 F, d]: an expert's gate rows, then its up rows (without a gate: [E, F, d]);
             # [E, d, F]
@@ -121,9 +143,13 @@ class RoutedExperts(FeedForward):
         if self.shared is not None:
             self.shared.load(tensors, ctx)
 
-    def forward(self, x):
+    def forward(self, x, lazy: bool = False):
         n, d = x.shape
         logits = self.router(x, out_dtype=torch.float32)
+        gate = None
+        if self.shared_gate:
+            total = self.experts + self.identity
+            logits, gate = logits[:, :total], logits[:, total:]
         tensor_cores = self._tensor_cores(x.dtype)
         ids, weights, pair_token, pair_place, meta, max_tiles, rows = ops.moe_route(
             logits, self.correction, None, self.experts, self.groups, self.keep_groups, self.top,
@@ -145,5 +171,8 @@ class RoutedExperts(FeedForward):
                                 gated=self.first)
                 ops.moe_product(hidden, self.down, y, meta, pair_token, max_tiles, gated=False)
         shared = self.shared.forward(x) if self.shared is not None else None
+        if lazy and self.hands_on_routed:
+            return RoutedSum(y, ids, weights, pair_place, shared, gate)
         out = torch.empty_like(x)
-        return ops.moe_combine(y, x, shared, ids, weights, pair_place, self.experts, out)
+        return ops.moe_combine(y, x, shared, ids, weights, pair_place, self.experts, out,
+                               shared_gate=gate)

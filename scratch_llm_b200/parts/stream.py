@@ -56,26 +56,62 @@ class Current:
 
 
 @dataclass
+class RoutedSum:
+    """A routed feed-forward's output that is not added up yet: token n's is ``sum_j weights[n, j]
+    * y[place[n, j]]`` over its choices, plus ``sigmoid(gate[n]) * shared[n]`` (without ``gate``:
+    plus ``shared[n]``; without ``shared``: nothing).  A norm that takes it (``takes_routed``)
+    adds it up in 32-bit while it reads the stream."""
+
+    y: torch.Tensor               # float32 [places, hidden]
+    ids: torch.Tensor             # int32 [tokens, top]
+    weights: torch.Tensor         # float32 [tokens, top]
+    place: torch.Tensor           # int32 [tokens * top], -1: no row
+    shared: torch.Tensor | None   # [tokens, hidden] in the compute dtype
+    gate: torch.Tensor | None     # float32 [tokens, 1]
+
+
+@dataclass
 class Terms:
     """What a layer leaves pending for the stream when it is a weighted sum of several branch
-    outputs: the stream is to receive ``sum(coef * tensor)``.  A norm that takes it
+    outputs: the stream is to receive ``sum(coef * tensor)``, plus a routed feed-forward's
+    output (``routed``, weight 1) where the norm takes one.  A norm that takes it
     (``takes_terms``) forms the sum in 32-bit while it reads the stream, so that neither the
     sum nor the products by the weights cost a pass or a rounding of their own."""
 
     items: tuple            # ((tensor [tokens, hidden], coefficient), ...)
+    routed: RoutedSum | None = None
 
     def scaled(self, factor: float) -> "Terms":
-        return Terms(tuple((t, c * factor) for t, c in self.items))
+        if self.routed is not None and factor != 1.0:
+            raise ValueError("a routed sum has no weight of its own")
+        return Terms(tuple((t, c * factor) for t, c in self.items), self.routed)
 
     @staticmethod
     def of(value, coef: float = 1.0) -> "Terms":
         """``coef * value`` as terms, whether ``value`` is a tensor or already a sum."""
+        if isinstance(value, RoutedSum):
+            return Terms((), value).scaled(coef)
         if isinstance(value, Terms):
             return value.scaled(coef)
         return Terms(((value, float(coef)),))
 
     def __add__(self, other: "Terms") -> "Terms":
-        return Terms(self.items + other.items)
+        if self.routed is not None and other.routed is not None:
+            raise ValueError("a sum takes one routed output")
+        return Terms(self.items + other.items, self.routed or other.routed)
+
+    def total(self) -> torch.Tensor:
+        """The sum as a 32-bit tensor, for looking into a model."""
+        out = sum(c * t.float() for t, c in self.items)
+        r = self.routed
+        if r is not None:
+            n, top = r.ids.shape
+            place = r.place.view(n, top).long()
+            rows = r.y[place.clamp(min=0)] * (place >= 0)[..., None]
+            out = out + (r.weights[..., None] * rows).sum(1)
+            if r.shared is not None:
+                out = out + r.shared.float() * (torch.sigmoid(r.gate) if r.gate is not None else 1.0)
+        return out
 
 
 class StreamSink:
