@@ -190,6 +190,34 @@ def tubevik_config(name: str):
                    {"type": "parallel", "mixer": both, "mlp": mlp}]})
 
 
+def deganex_config(name: str):
+    """The Deganex design at the sizes of COMPARE_SIZES: a state-space layer (twice the width in
+    heads of 64, state 128), latent attention (as many heads, the head size as the unrotated
+    part, a rotated part of 64, a latent of 192: the cached vector has 256 entries, the largest
+    the tensor-core attention kernels take), a matrix memory (keys of 256, values of 512, one
+    head per 512 of the width) and latent attention again; every layer with a routed
+    feed-forward of 16 experts and a gated shared one, each a quarter of the dense size, of which
+    a token uses 3 and the shared one: as much as the dense feed-forward."""
+    from scratch_llm_b200.config import config_from_dict
+
+    z = COMPARE_SIZES[name]
+    d = z["width"]
+    mlp = {"kind": "moe", "expert": {"ff": z["ff"] // 4}, "router": {"experts": 16, "top": 3},
+           "shared": {"ff": z["ff"] // 4}}
+    latent = {"type": "latent_attention", "mlp": mlp, "mixer": {
+        "heads": z["heads"], "dim": z["dim"], "rot_dim": 64, "vdim": z["dim"], "kv_rank": 192,
+        "scale": (z["dim"] + 64) ** -0.5, "rot": {"base": 1000000.0, "dims": 64}}}
+    state_space = {"type": "mamba2", "mlp": mlp, "mixer": {
+        "heads": 2 * d // 64, "vdim": 64, "state": 128, "groups": 4, "conv": 4, "norm_groups": 4}}
+    memory = {"type": "mlstm", "mlp": mlp, "mixer": {
+        "heads": d // 512, "dim": 256, "vdim": 512, "gate_cap": 20.0}}
+    return config_from_dict({
+        "architecture": "Deganex", "vocab": z["vocab"], "width": d, "norm": {"eps": 1e-5},
+        "logit_softcap": 25.0, "max_position": 8192,
+        "embedding": {"bigram": {"buckets": 65521, "mul_prev": 4099, "mul_cur": 257}},
+        "layers": [state_space, latent, memory, latent]})
+
+
 #: low ranks that only a model's tensors say (a size of -1 in a parameter's shape): random
 #: weights are drawn with this one
 RANDOM_LOW_RANK = 64
@@ -228,12 +256,14 @@ def engine_of(cfg, capacity_tokens: int, max_requests: int, page_size: int):
 
 
 def compare_main(args) -> int:
-    """--compare nilevik | vobosun | titedra | tubevik: prefill and decode throughput of that design beside
+    """--compare nilevik | vobosun | titedra | tubevik | deganex: prefill and decode throughput of that design beside
     the engine's other models of equal size (for Vobosun: Nilevik, the closest one, a hybrid of
     attention and a delta rule with normed branch outputs, and the Llama-style model; for
     Titedra: Vobosun, the closest one, with norms around every branch, a partly rotated
     attention and routed experts, and the Llama-style model; for Tubevik: Nilevik, the closest one, likewise a hybrid of windowed
-    attention and a gated delta rule, and the Llama-style model), at the sizes of COMPARE_SIZES.
+    attention and a gated delta rule, and the Llama-style model; for Deganex: Titedra, the closest
+    one, with latent attention and routed experts, Nilevik for its recurrence, and the
+    Llama-style model), at the sizes of COMPARE_SIZES.
     One JSON line."""
     import torch
 
@@ -263,6 +293,10 @@ def compare_main(args) -> int:
                                            "dense")
                 archs = [("titedra", titedra_config(name))] + \
                     [a for a in archs if a[0] != "nilevik"]
+            if args.compare == "deganex":
+                entry["deganex_layers"] = ("state space, latent attention, matrix memory, latent "
+                                           "attention, each + routed with a shared expert")
+                archs[:0] = [("deganex", deganex_config(name)), ("titedra", titedra_config(name))]
             for arch, cfg in archs:
                 llm = engine_of(cfg, capacity, args.batch + 1, args.page_size)
                 with ClockSampler(0) as clk:
@@ -424,7 +458,7 @@ def main() -> int:
                     help="layer sizes (the default is the configuration the metric is quoted on)")
     ap.add_argument("--serve", type=int, default=0, metavar="N",
                     help="also run the continuous-batching workload with N requests")
-    ap.add_argument("--compare", default=None, choices=["nilevik", "vobosun", "titedra", "tubevik"],
+    ap.add_argument("--compare", default=None, choices=["nilevik", "vobosun", "titedra", "tubevik", "deganex"],
                     help="instead of the headline workload: prefill and decode throughput of "
                          "this design beside the Llama-style model of equal size")
     ap.add_argument("--compare-sizes", default=None, choices=sorted(COMPARE_SIZES),

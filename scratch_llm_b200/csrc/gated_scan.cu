@@ -49,12 +49,20 @@ struct ScanArgs {
     const float* skip;                   // [H] or null
     float scale;
     int H, G, N, V, VX;
+    int vec4;                            // rows of q and k allow reads of four elements
     int min_chunked;                     // rows of at least so many tokens are the chunk kernels'
     // chunk kernels only
     float* dS;                           // [slots of chunks, H, VX, N]
     float* decay;                        // [slots of chunks, H]: L of the chunk's last token
     int n_rows;
 };
+
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+    return make_float4(__low2float(h[0]), __high2float(h[0]), __low2float(h[1]), __high2float(h[1]));
+}
 
 // ------------------------------------------------------------------------ token by token
 
@@ -103,11 +111,22 @@ __global__ void __launch_bounds__(256) gated_scan_kernel(const ScanArgs a, int t
     for (int c0 = 0; c0 < n_new; c0 += tokens_staged) {
         const int nt = min(tokens_staged, n_new - c0);
         if (c0) __syncthreads();               // the previous chunk is no longer read
-        for (int i = tid; i < nt * NP; i += 256) {
-            const int t = i / NP, e = i - t * NP;
-            const int64_t n = t0 + c0 + t;
-            ks[i] = e < N ? to_float(k[n * a.ldk + e]) : 0.f;
-            qs[i] = e < N ? to_float(q[n * a.ldq + e]) : 0.f;
+        if (quads && a.vec4) {                 // four elements of a row at a time
+            const int per = N / 4;
+#pragma unroll 4
+            for (int i = tid; i < nt * per; i += 256) {
+                const int t = i / per, e = (i - t * per) * 4;
+                const int64_t n = t0 + c0 + t;
+                *reinterpret_cast<float4*>(ks + t * NP + e) = load4(k + n * a.ldk + e);
+                *reinterpret_cast<float4*>(qs + t * NP + e) = load4(q + n * a.ldq + e);
+            }
+        } else {
+            for (int i = tid; i < nt * NP; i += 256) {
+                const int t = i / NP, e = i - t * NP;
+                const int64_t n = t0 + c0 + t;
+                ks[i] = e < N ? to_float(k[n * a.ldk + e]) : 0.f;
+                qs[i] = e < N ? to_float(q[n * a.ldq + e]) : 0.f;
+            }
         }
         for (int i = tid; i < nt * COLS; i += 256) {
             const int t = i / COLS, j = col0 + i - t * COLS;
@@ -120,7 +139,7 @@ __global__ void __launch_bounds__(256) gated_scan_kernel(const ScanArgs a, int t
         __syncthreads();
         for (int t = 0; t < nt; ++t) {
             const float decay = as[t], value = vs[t * COLS + col - col0], bv = bs[t] * value;
-            float acc = 0.f;
+            float part[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
             for (int i = 0; i < QPL; ++i) {
                 const int e = (i * LPC + sub) * 4;
@@ -131,12 +150,13 @@ __global__ void __launch_bounds__(256) gated_scan_kernel(const ScanArgs a, int t
                     S[4 * i + 1] = fmaf(decay, S[4 * i + 1], bv * kk.y);
                     S[4 * i + 2] = fmaf(decay, S[4 * i + 2], bv * kk.z);
                     S[4 * i + 3] = fmaf(decay, S[4 * i + 3], bv * kk.w);
-                    acc = fmaf(S[4 * i], qq.x, acc);
-                    acc = fmaf(S[4 * i + 1], qq.y, acc);
-                    acc = fmaf(S[4 * i + 2], qq.z, acc);
-                    acc = fmaf(S[4 * i + 3], qq.w, acc);
+                    part[0] = fmaf(S[4 * i], qq.x, part[0]);
+                    part[1] = fmaf(S[4 * i + 1], qq.y, part[1]);
+                    part[2] = fmaf(S[4 * i + 2], qq.z, part[2]);
+                    part[3] = fmaf(S[4 * i + 3], qq.w, part[3]);
                 }
             }
+            float acc = (part[0] + part[1]) + (part[2] + part[3]);
 #pragma unroll
             for (int o = LPC / 2; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
             if (sub == 0 && live) {
@@ -257,24 +277,28 @@ __device__ __forceinline__ void chunk_gates(const ScanArgs& a, int64_t n0, int n
     Ls[2 * lane + 1] = before + x0 + x1;
 }
 
-// `rows` rows of N bfloat16 (N % 8 == 0, 16-byte aligned) into shared memory, row stride ld;
-// rows from nt on are zero.
+// TC rows of N bfloat16 (N % 8 == 0, 16-byte aligned) into shared memory, row stride ld; rows from
+// nt on are zero.
 __device__ __forceinline__ void stage_rows(bf16* dst, int ld, const bf16* src, int64_t lds, int nt,
                                            int N) {
-    const int units = N / 8;
-    for (int i = threadIdx.x; i < TC * units; i += blockDim.x) {
-        const int t = i / units, u = i - t * units;
+    const int units = N / 8, dt = blockDim.x / units, du = blockDim.x - dt * units;
+    int t = threadIdx.x / units, u = threadIdx.x - t * units;
+#pragma unroll 4
+    for (; t < TC;) {
         uint4 x = make_uint4(0u, 0u, 0u, 0u);
         if (t < nt) x = *reinterpret_cast<const uint4*>(src + (int64_t)t * lds + u * 8);
         *reinterpret_cast<uint4*>(dst + t * ld + u * 8) = x;
+        t += dt;
+        u += du;
+        if (u >= units) { u -= units; ++t; }
     }
 }
 
-// dS of one chunk and head, columns [v0, v0 + cols).  128 threads: the 16-row tiles of S's columns
-// (m) against N (n), every warp a quarter of N's 8-wide tiles; the sum runs over the tokens.
-__global__ void __launch_bounds__(128) chunk_state_kernel(const ScanArgs a) {
+// dS of one chunk and head, columns [v0, v0 + cols).  256 threads: the 16-row tiles of S's columns
+// (m) against N (n), every warp an eighth of N's 8-wide tiles; the sum runs over the tokens.
+__global__ void __launch_bounds__(256) chunk_state_kernel(const ScanArgs a) {
     extern __shared__ __align__(16) unsigned char raw[];
-    __shared__ float Ls[TC], bs[TC];
+    __shared__ float Ls[TC], bs[TC], ws[TC];
     pdl_wait();
     pdl_trigger();
     int row, t0, c0, n_new;
@@ -298,32 +322,48 @@ __global__ void __launch_bounds__(128) chunk_state_kernel(const ScanArgs a) {
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     if (tid == 0 && blockIdx.z == 0) a.decay[(int64_t)blockIdx.x * H + head] = L_last;
     const int m_tiles = (cols + 15) / 16;
-    for (int i = tid; i < TC * m_tiles * 8; i += 128) {    // pairs of columns
-        const int t = i / (m_tiles * 8), j = (i - t * m_tiles * 8) * 2;
-        float x = 0.f, y = 0.f;
-        if (t < nt) {
-            const float w = expf(L_last - Ls[t]) * bs[t];
-            const int c = v0 + j;
-            x = j < cols ? (c < V ? to_float(v[(int64_t)t * a.ldv + c]) : 1.f) * w : 0.f;
-            y = j + 1 < cols ? (c + 1 < V ? to_float(v[(int64_t)t * a.ldv + c + 1]) : 1.f) * w : 0.f;
-        }
-        uint32_t part[PARTS];
-        split2(x, y, part);
+    if (tid < TC) ws[tid] = expf(L_last - Ls[tid]) * bs[tid];
+    __syncthreads();
+    for (int jp = lane; jp < m_tiles * 8; jp += 32) {      // pairs of columns (V is even)
+        const int j = jp * 2, c = v0 + j;
 #pragma unroll
-        for (int p = 0; p < PARTS; ++p)
-            *reinterpret_cast<uint32_t*>(vs + (p * TC + t) * LDV + j) = part[p];
+        for (int i = 0; i < TC / 8; ++i) {
+            const int t = warp + i * 8;
+            float x = 0.f, y = 0.f;
+            if (t < nt && j < cols) {
+                const float w = ws[t];
+                x = w;                                     // the column of ones, and nothing behind
+                if (c < V) {
+                    const __nv_bfloat162 h =
+                        *reinterpret_cast<const __nv_bfloat162*>(v + (int64_t)t * a.ldv + c);
+                    x = __low2float(h) * w;
+                    y = __high2float(h) * w;
+                }
+            }
+            uint32_t part[PARTS];
+            split2(x, y, part);
+#pragma unroll
+            for (int p = 0; p < PARTS; ++p)
+                *reinterpret_cast<uint32_t*>(vs + (p * TC + t) * LDV + j) = part[p];
+        }
     }
     __syncthreads();
     float* dst = a.dS + (((int64_t)blockIdx.x * H + head) * a.VX + v0) * N;
     const int n_tiles = N / 8;
-    // a warp's share of the n tiles, two at a time
-    for (int nb = warp * 2; nb < n_tiles; nb += 8) {
-        uint32_t bfrag[TC / 16][4];      // per 16 tokens: tiles nb and nb + 1
+    // warps w and w + 4: four of the n tiles at a time, every other of the m tiles
+    for (int nb = (warp & 3) * 4; nb < n_tiles; nb += 16) {
+        const bool wide = nb + 2 < n_tiles;                // (the number of n tiles is even)
+        uint32_t bfrag[TC / 16][8];      // per 16 tokens: tiles nb .. nb + 3
 #pragma unroll
-        for (int kt = 0; kt < TC / 16; ++kt)
-            ldsm4_t(bfrag[kt], smem_addr(ks + (kt * 16 + (lane & 15)) * ldk + nb * 8 + (lane >> 4) * 8));
-        for (int mt = 0; mt < m_tiles; ++mt) {
-            float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+        for (int kt = 0; kt < TC / 16; ++kt) {
+            const bf16* at = ks + (kt * 16 + (lane & 15)) * ldk + nb * 8 + (lane >> 4) * 8;
+            ldsm4_t(bfrag[kt], smem_addr(at));
+            if (wide) ldsm4_t(bfrag[kt] + 4, smem_addr(at + 16));
+        }
+        for (int mt = warp >> 2; mt < m_tiles; mt += 2) {
+            float acc[4][4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) acc[u][0] = acc[u][1] = acc[u][2] = acc[u][3] = 0.f;
 #pragma unroll
             for (int p = PARTS - 1; p >= 0; --p)           // small parts first
 #pragma unroll
@@ -336,17 +376,19 @@ __global__ void __launch_bounds__(128) chunk_state_kernel(const ScanArgs a) {
                                           mt * 16 + (blk & 1) * 8));
                     mma_bf16(acc[0], af, bfrag[kt]);
                     mma_bf16(acc[1], af, bfrag[kt] + 2);
+                    if (wide) {
+                        mma_bf16(acc[2], af, bfrag[kt] + 4);
+                        mma_bf16(acc[3], af, bfrag[kt] + 6);
+                    }
                 }
-            const int m = mt * 16 + (lane >> 2), n = nb * 8 + (lane & 3) * 2;
+            const int m = mt * 16 + (lane >> 2);
+            float* d = dst + (int64_t)m * N + nb * 8 + (lane & 3) * 2;
 #pragma unroll
-            for (int u = 0; u < 2; ++u) {
+            for (int u = 0; u < 4; ++u) {
                 if (nb + u >= n_tiles) break;
-                if (m < cols)
-                    *reinterpret_cast<float2*>(dst + (int64_t)m * N + n + u * 8) =
-                        make_float2(acc[u][0], acc[u][1]);
+                if (m < cols) *reinterpret_cast<float2*>(d + u * 8) = make_float2(acc[u][0], acc[u][1]);
                 if (m + 8 < cols)
-                    *reinterpret_cast<float2*>(dst + (int64_t)(m + 8) * N + n + u * 8) =
-                        make_float2(acc[u][2], acc[u][3]);
+                    *reinterpret_cast<float2*>(d + 8 * N + u * 8) = make_float2(acc[u][2], acc[u][3]);
             }
         }
     }
@@ -354,7 +396,7 @@ __global__ void __launch_bounds__(128) chunk_state_kernel(const ScanArgs a) {
 
 // The states at the chunks' starts, in place of the chunks' own dS, and the row's final state
 // into its slot.  A thread per four elements; grid (ceil(VX N / 4 / 256), H, rows).
-constexpr int PASS_AHEAD = 4;
+constexpr int PASS_AHEAD = 8;
 __global__ void __launch_bounds__(256) chunk_pass_kernel(const ScanArgs a) {
     pdl_wait();
     pdl_trigger();
@@ -392,9 +434,14 @@ __global__ void __launch_bounds__(256) chunk_pass_kernel(const ScanArgs a) {
     *home = S;
 }
 
-// The read-outs of one chunk and head, columns [v0, v0 + cols).  128 threads: warp w has the
-// chunk's tokens 16 w .. 16 w + 15.
-__global__ void __launch_bounds__(128) chunk_out_kernel(const ScanArgs a) {
+// The read-outs of one chunk and head, columns [v0, v0 + cols).  256 threads: warps w and w + 4 have
+// the chunk's tokens 16 w .. 16 w + 15, and half of the columns' tiles each.  The keys, queries and
+// state go through shared memory in slabs of KB elements of N.
+constexpr int KB = 64, LDB = KB + 8;
+constexpr int OT = (VT / 8 + 1) / 2;                       // column tiles of a warp
+constexpr int OUT_LDV = VT + 16;
+constexpr size_t OUT_SMEM = ((size_t)(2 * TC + PARTS * VT) * LDB + (size_t)TC * OUT_LDV) * sizeof(bf16);
+__global__ void __launch_bounds__(256, 3) chunk_out_kernel(const ScanArgs a) {
     extern __shared__ __align__(16) unsigned char raw[];
     __shared__ float Ls[TC], bs[TC];
     pdl_wait();
@@ -408,36 +455,19 @@ __global__ void __launch_bounds__(128) chunk_out_kernel(const ScanArgs a) {
     const bool last_block = blockIdx.z == gridDim.z - 1;
     const int cols = last_block ? a.VX - v0 : VB;
     const int n_tiles = (cols + 7) / 8;                    // up to VT / 8 = 9
-    const int ldk = N + 8;
-    constexpr int LDV = VT + 16;                           // 88
-    bf16* ks = reinterpret_cast<bf16*>(raw);               // [TC][ldk]
-    bf16* qs = ks + TC * ldk;                              // [TC][ldk]
-    bf16* ss = qs + TC * ldk;                              // [PARTS][VT][ldk]: the state's columns
-    bf16* vs = ss + PARTS * VT * ldk;                      // [TC][LDV]
+    constexpr int LDV = OUT_LDV;
+    bf16* ks = reinterpret_cast<bf16*>(raw);               // [TC][LDB]
+    bf16* qs = ks + TC * LDB;                              // [TC][LDB]
+    bf16* ss = qs + TC * LDB;                              // [PARTS][VT][LDB]: the state's columns
+    bf16* vs = ss + PARTS * VT * LDB;                      // [TC][LDV]
     const int g = head / (H / a.G);
     const bf16* k = reinterpret_cast<const bf16*>(a.k) + n0 * a.ldk + (int64_t)g * N;
     const bf16* q = reinterpret_cast<const bf16*>(a.q) + n0 * a.ldq + (int64_t)g * N;
     const bf16* v = reinterpret_cast<const bf16*>(a.v) + n0 * a.ldv + (int64_t)head * V;
+    const float* s0 = a.dS + (((int64_t)blockIdx.x * H + head) * a.VX + v0) * N;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     chunk_gates(a, n0, nt, head, Ls, bs);
-    stage_rows(ks, ldk, k, a.ldk, nt, N);
-    stage_rows(qs, ldk, q, a.ldq, nt, N);
-    {   // S0's columns, split; zero columns up to a whole tile
-        const float* s0 = a.dS + (((int64_t)blockIdx.x * H + head) * a.VX + v0) * N;
-        const int per = N / 4;
-        for (int i = tid; i < n_tiles * 8 * per; i += 128) {
-            const int j = i / per, e = (i - j * per) * 4;
-            float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (j < cols) x = *reinterpret_cast<const float4*>(s0 + (int64_t)j * N + e);
-            uint32_t lo[PARTS], hi[PARTS];
-            split2(x.x, x.y, lo);
-            split2(x.z, x.w, hi);
-#pragma unroll
-            for (int p = 0; p < PARTS; ++p)
-                *reinterpret_cast<uint2*>(ss + (p * VT + j) * ldk + e) = make_uint2(lo[p], hi[p]);
-        }
-    }
-    for (int i = tid; i < TC * n_tiles; i += 128) {        // eight values at a time
+    for (int i = tid; i < TC * n_tiles; i += 256) {        // eight values at a time
         const int t = i / n_tiles, j = (i - t * n_tiles) * 8;
         alignas(16) bf16 x[8];
         if (t < nt && v0 + j + 8 <= V) {
@@ -452,87 +482,139 @@ __global__ void __launch_bounds__(128) chunk_out_kernel(const ScanArgs a) {
         }
         *reinterpret_cast<uint4*>(vs + t * LDV + j) = *reinterpret_cast<const uint4*>(x);
     }
-    __syncthreads();
-    float o[VT / 8][4];
+    const int m0 = (warp & 3) * 16, side = warp >> 2;
+    const int first = side ? (n_tiles + 1) / 2 : 0;        // this warp's column tiles
+    const int mine = side ? n_tiles / 2 : (n_tiles + 1) / 2;
+    float o[OT][4];
 #pragma unroll
-    for (int j = 0; j < VT / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-    float w[TC / 8][4];                                    // k_s . q_t, then the weights
+    for (int j = 0; j < OT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+    // k_s . q_t of this warp's tokens t and half of the tokens s: the groups of 16 with the
+    // numbers side and side + 2
+    float w[2][2][4];
 #pragma unroll
-    for (int j = 0; j < TC / 8; ++j) w[j][0] = w[j][1] = w[j][2] = w[j][3] = 0.f;
-    const int m0 = warp * 16;
-    for (int kt = 0; kt < N / 16; ++kt) {
-        uint32_t af[4];
-        ldsm4(af, smem_addr(qs + (m0 + (lane & 15)) * ldk + kt * 16 + (lane >> 4) * 8));
+    for (int i = 0; i < 2; ++i)
 #pragma unroll
-        for (int j = 0; j < TC / 8; j += 2) {              // keys of tokens 8 j .. 8 j + 15
-            if (j * 8 > m0 + 15) break;                    // later than this warp's tokens
-            uint32_t bf[4];
-            ldsm4(bf, smem_addr(ks + (j * 8 + (lane >> 4) * 8 + (lane & 7)) * ldk + kt * 16 +
-                                ((lane >> 3) & 1) * 8));
-            mma_bf16(w[j], af, bf);
-            mma_bf16(w[j + 1], af, bf + 2);
-        }
+        for (int u = 0; u < 4; ++u) w[i][0][u] = w[i][1][u] = 0.f;
+    for (int kb = 0; kb < N; kb += KB) {
+        const int width = min(KB, N - kb);
+        if (kb) __syncthreads();                           // the previous slab is no longer read
+        stage_rows(ks, LDB, k + kb, a.ldk, nt, width);
+        stage_rows(qs, LDB, q + kb, a.ldq, nt, width);
+        {   // S0's columns, split; zero columns up to a whole tile
+            const int e = (tid & 15) * 4;
+            if (e < width) {
 #pragma unroll
-        for (int p = PARTS - 1; p >= 0; --p)
+                for (int i = 0; i < VT / 16 + 1; ++i) {
+                    const int j = (tid >> 4) + i * 16;
+                    if (j >= n_tiles * 8) break;
+                    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+                    if (j < cols) x = *reinterpret_cast<const float4*>(s0 + (int64_t)j * N + kb + e);
+                    uint32_t lo[PARTS], hi[PARTS];
+                    split2(x.x, x.y, lo);
+                    split2(x.z, x.w, hi);
 #pragma unroll
-            for (int j = 0; j < VT / 8; ++j) {
-                if (j >= n_tiles) break;
-                uint32_t bf[2];
-                ldsm2(bf, smem_addr(ss + (p * VT + j * 8 + (lane & 7)) * ldk + kt * 16 +
-                                    ((lane >> 3) & 1) * 8));
-                mma_bf16(o[j], af, bf);
+                    for (int p = 0; p < PARTS; ++p)
+                        *reinterpret_cast<uint2*>(ss + (p * VT + j) * LDB + e) =
+                            make_uint2(lo[p], hi[p]);
+                }
             }
+        }
+        __syncthreads();
+        for (int kt = 0; kt < width / 16; ++kt) {
+            uint32_t af[4];
+            ldsm4(af, smem_addr(qs + (m0 + (lane & 15)) * LDB + kt * 16 + (lane >> 4) * 8));
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const int sg = (side + 2 * i) * 16;
+                if (sg > m0) break;                       // later than this warp's tokens
+                uint32_t bf[4];
+                ldsm4(bf, smem_addr(ks + (sg + (lane >> 4) * 8 + (lane & 7)) * LDB + kt * 16 +
+                                    ((lane >> 3) & 1) * 8));
+                mma_bf16(w[i][0], af, bf);
+                mma_bf16(w[i][1], af, bf + 2);
+            }
+#pragma unroll
+            for (int p = PARTS - 1; p >= 0; --p)
+#pragma unroll
+                for (int j = 0; j < OT; j += 2) {          // two tiles a load
+                    if (j >= mine) break;
+                    uint32_t bf[4];
+                    ldsm4(bf, smem_addr(ss + (p * VT + (first + j + (lane >> 4)) * 8 + (lane & 7)) * LDB +
+                                        kt * 16 + ((lane >> 3) & 1) * 8));
+                    mma_bf16(o[j], af, bf);
+                    if (j + 1 < OT && j + 1 < mine) mma_bf16(o[j + 1], af, bf + 2);
+                }
+        }
     }
     const int ta = m0 + (lane >> 2), tb = ta + 8;          // this thread's two tokens
-    const float La = Ls[ta], Lb = Ls[tb], ea = expf(La), eb = expf(Lb);
+    const float La = Ls[ta], Lb = Ls[tb], ea = __expf(La), eb = __expf(Lb);
 #pragma unroll
-    for (int j = 0; j < VT / 8; ++j) {
+    for (int j = 0; j < OT; ++j) {
         o[j][0] *= ea; o[j][1] *= ea;
         o[j][2] *= eb; o[j][3] *= eb;
     }
+    // the weights, split, into the state's place: [PARTS][TC][LDB]
+    __syncthreads();
+    bf16* ps = ss;
 #pragma unroll
-    for (int j = 0; j < TC / 8; ++j) {
-        const int s = j * 8 + (lane & 3) * 2;
+    for (int i = 0; i < 2; ++i) {
+        const int sg = (side + 2 * i) * 16;
+        if (sg > m0) break;
 #pragma unroll
-        for (int u = 0; u < 2; ++u) {
-            const float L = Ls[s + u], b = bs[s + u];
-            w[j][u] = s + u <= ta ? w[j][u] * expf(La - L) * b : 0.f;
-            w[j][2 + u] = s + u <= tb ? w[j][2 + u] * expf(Lb - L) * b : 0.f;
+        for (int h = 0; h < 2; ++h) {
+            const int s = sg + h * 8 + (lane & 3) * 2;
+            const float L0 = Ls[s], L1 = Ls[s + 1], b0 = bs[s], b1 = bs[s + 1];
+            const float* x = w[i][h];
+            uint32_t pa[PARTS], pb[PARTS];
+            split2(s <= ta ? x[0] * __expf(La - L0) * b0 : 0.f,
+                   s + 1 <= ta ? x[1] * __expf(La - L1) * b1 : 0.f, pa);
+            split2(s <= tb ? x[2] * __expf(Lb - L0) * b0 : 0.f,
+                   s + 1 <= tb ? x[3] * __expf(Lb - L1) * b1 : 0.f, pb);
+#pragma unroll
+            for (int p = 0; p < PARTS; ++p) {
+                *reinterpret_cast<uint32_t*>(ps + (p * TC + ta) * LDB + s) = pa[p];
+                *reinterpret_cast<uint32_t*>(ps + (p * TC + tb) * LDB + s) = pb[p];
+            }
         }
     }
+    __syncthreads();
 #pragma unroll
     for (int kt = 0; kt < TC / 16; ++kt) {                 // tokens s of 16
-        if (kt * 16 > m0 + 15) break;
-        uint32_t pa[4][PARTS];
-        split2(w[2 * kt][0], w[2 * kt][1], pa[0]);
-        split2(w[2 * kt][2], w[2 * kt][3], pa[1]);
-        split2(w[2 * kt + 1][0], w[2 * kt + 1][1], pa[2]);
-        split2(w[2 * kt + 1][2], w[2 * kt + 1][3], pa[3]);
+        if (kt * 16 > m0) break;
+        uint32_t af[PARTS][4];
 #pragma unroll
-        for (int j = 0; j < VT / 8; ++j) {
-            if (j >= n_tiles) break;
+        for (int p = 0; p < PARTS; ++p)
+            ldsm4(af[p], smem_addr(ps + (p * TC + m0 + (lane & 15)) * LDB + kt * 16 + (lane >> 4) * 8));
+#pragma unroll
+        for (int j = 0; j < OT; ++j) {
+            if (j >= mine) break;
             uint32_t bf[2];
-            ldsm2_t(bf, smem_addr(vs + (kt * 16 + (lane & 15)) * LDV + j * 8));
+            ldsm2_t(bf, smem_addr(vs + (kt * 16 + (lane & 15)) * LDV + (first + j) * 8));
 #pragma unroll
-            for (int p = PARTS - 1; p >= 0; --p) {
-                const uint32_t af[4] = {pa[0][p], pa[1][p], pa[2][p], pa[3][p]};
-                mma_bf16(o[j], af, bf);
-            }
+            for (int p = PARTS - 1; p >= 0; --p) mma_bf16(o[j], af[p], bf);
         }
     }
     const float skip = a.skip ? a.skip[head] : 0.f;
 #pragma unroll
-    for (int j = 0; j < VT / 8; ++j) {
-        if (j >= n_tiles) break;
+    for (int j = 0; j < OT; ++j) {
+        if (j >= mine) break;
+        const int jc = (first + j) * 8 + (lane & 3) * 2, c = v0 + jc;
 #pragma unroll
-        for (int u = 0; u < 4; ++u) {
-            const int t = u < 2 ? ta : tb, jc = j * 8 + (lane & 3) * 2 + (u & 1), c = v0 + jc;
+        for (int u = 0; u < 2; ++u) {
+            const int t = u ? tb : ta;
             if (t >= nt || c >= a.VX) continue;
-            const float x = o[j][u] * a.scale;
-            if (c >= V) a.ones_out[(n0 + t) * H + head] = x;
-            else
-                a.out[(n0 + t) * H * V + (int64_t)head * V + c] =
-                    skip != 0.f ? fmaf(skip, to_float(vs[t * LDV + jc]), x) : x;
+            float x = o[j][2 * u] * a.scale, y = o[j][2 * u + 1] * a.scale;
+            if (c >= V) {                                  // (V is even: the column of ones is x)
+                a.ones_out[(n0 + t) * H + head] = x;
+                continue;
+            }
+            if (skip != 0.f) {
+                const __nv_bfloat162 h = *reinterpret_cast<const __nv_bfloat162*>(vs + t * LDV + jc);
+                x = fmaf(skip, __low2float(h), x);
+                y = fmaf(skip, __high2float(h), y);
+            }
+            *reinterpret_cast<float2*>(a.out + (n0 + t) * H * V + (int64_t)head * V + c) =
+                make_float2(x, y);
         }
     }
 }
@@ -552,22 +634,23 @@ SLLM_EXPORT int sllm_gated_scan_chunks_fit(int N, int V) {
 // float [slots, H, V + ones, N]; out: float [n_tokens, H V]; ones_out: float [n_tokens, H] (ones
 // only); skip: float [H] or null.  chunked: rows of at least min_chunked tokens take the chunk
 // kernels, with the scratch dS float [n_tokens / 64 + n_rows + 1, H, V + ones, N] and decay float
-// [the same, H]; else every row is walked token by token.  longest: the most tokens a row brings (an
-// upper bound).
+// [the same, H]; else every row is walked token by token.  shortest / longest: bounds of the tokens
+// a row brings.
 SLLM_EXPORT int sllm_gated_scan(const void* q, int64_t ldq, const void* k, int64_t ldk,
                                 const void* v, int64_t ldv, const float* log_a, const float* b,
                                 float* state, const int* row_start, const int* row_slot,
                                 float* out, float* ones_out, const float* skip, float scale,
                                 int n_tokens, int n_rows, int H, int G, int N, int V, int ones,
-                                int chunked, int min_chunked, int longest, float* dS, float* decay,
-                                int dtype, cudaStream_t stream) {
+                                int chunked, int min_chunked, int shortest, int longest, float* dS,
+                                float* decay, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0 || n_rows <= 0) return 0;
     if (H < 1 || G < 1 || H % G || N < 1 || N > 1024 || V < 1 || ones < 0 || ones > 1 ||
         (ones && !ones_out) || ldq < (int64_t)G * N || ldk < (int64_t)G * N ||
         ldv < (int64_t)H * V || H > 65535 || n_rows > 65535 || dtype < 0 || dtype > 1)
         return (int)cudaErrorInvalidValue;
+    const int vec4 = !((ldq | ldk | N) & 3) && !(((uintptr_t)q | (uintptr_t)k) & 15);
     ScanArgs a = {q, ldq, k, ldk, v, ldv, log_a, b, state, row_start, row_slot, out, ones_out, skip,
-                  scale, H, G, N, V, V + ones, 0x7fffffff, dS, decay, n_rows};
+                  scale, H, G, N, V, V + ones, vec4, 0x7fffffff, dS, decay, n_rows};
     if ((N & 3) == 0 && ((uintptr_t)state & 15)) return (int)cudaErrorInvalidValue;
     if (chunked) {
         if (dtype != 1 || !dS || !decay || min_chunked < 1 || !sllm_gated_scan_chunks_fit(N, V) ||
@@ -578,34 +661,32 @@ SLLM_EXPORT int sllm_gated_scan(const void* q, int64_t ldq, const void* k, int64
         const int slots = n_tokens / TC + n_rows + 1;
         const int blocks_v = (V + VB - 1) / VB;
         const size_t smem_state = ((size_t)TC * (N + 8) + (size_t)PARTS * TC * 88) * sizeof(bf16);
-        const size_t smem_out =
-            ((size_t)(2 * TC + PARTS * VT) * (N + 8) + (size_t)TC * (VT + 16)) * sizeof(bf16);
         static bool ready = false;
         if (!ready) {
-            const int top = 227 * 1024 - 1024;
-            cudaError_t e = cudaFuncSetAttribute(chunk_state_kernel,
-                                                 cudaFuncAttributeMaxDynamicSharedMemorySize, top);
+            cudaError_t e = cudaFuncSetAttribute(
+                chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - 1024);
             if (e == cudaSuccess)
                 e = cudaFuncSetAttribute(chunk_out_kernel,
-                                         cudaFuncAttributeMaxDynamicSharedMemorySize, top);
+                                         cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         (int)OUT_SMEM);
             if (e != cudaSuccess) return (int)e;
             ready = true;
         }
         const int64_t quads = (int64_t)a.VX * N / 4;
-        cudaError_t e = sllm_launch_pdl(chunk_state_kernel, dim3(slots, H, blocks_v), dim3(128),
+        cudaError_t e = sllm_launch_pdl(chunk_state_kernel, dim3(slots, H, blocks_v), dim3(256),
                                         smem_state, stream, a);
         if (e != cudaSuccess) return (int)e;
         e = sllm_launch_pdl(chunk_pass_kernel, dim3((unsigned)((quads + 255) / 256), H, n_rows),
                             dim3(256), 0, stream, a);
         if (e != cudaSuccess) return (int)e;
-        e = sllm_launch_pdl(chunk_out_kernel, dim3(slots, H, blocks_v), dim3(128), smem_out, stream,
+        e = sllm_launch_pdl(chunk_out_kernel, dim3(slots, H, blocks_v), dim3(256), OUT_SMEM, stream,
                             a);
         if (e != cudaSuccess) return (int)e;
     }
     const int NP = (N + 3) / 4 * 4;
     int limit = longest > 0 ? longest : 32;
     if (chunked && limit > min_chunked - 1) limit = min_chunked - 1;
-    if (limit < 1) return 0;
+    if (limit < 1 || (chunked && shortest >= min_chunked)) return 0;   // nothing left
 #define SLLM_SCAN(T, LPC, EPL)                                                                     \
     do {                                                                                           \
         constexpr int cols = 8 * 32 / LPC;                                                         \

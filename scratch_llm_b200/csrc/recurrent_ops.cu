@@ -140,6 +140,71 @@ __global__ void conv_silu_vec_kernel(const __nv_bfloat16* __restrict__ x, int64_
     }
 }
 
+// Long steps: a thread takes 8 consecutive channels of CONV_RUN consecutive tokens, so that the
+// taps are read once for all of them and every input once (the last K - 1 inputs stay in registers;
+// at the start of the run, and where another row starts within it, they are read).  The
+// arithmetic and its order are the scalar kernel's.
+constexpr int CONV_RUN = 8;
+template <int K>
+__global__ void __launch_bounds__(128)
+conv_silu_run_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx,
+                     const float* __restrict__ taps_t, const float* __restrict__ bias,
+                     const __nv_bfloat16* __restrict__ state, const int* __restrict__ token_row,
+                     const int* __restrict__ row_start, const int* __restrict__ row_slot,
+                     __nv_bfloat16* __restrict__ out, int C, int n_tokens) {
+    pdl_wait();
+    pdl_trigger();
+    typedef __nv_bfloat16 bf16;
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+    if (c >= C) return;
+    float tp[K][8], b[8];
+#pragma unroll
+    for (int j = 0; j < K; ++j) {
+        Vec<float>::load(taps_t + (int64_t)j * C + c, tp[j]);
+        Vec<float>::load(taps_t + (int64_t)j * C + c + 4, tp[j] + 4);
+    }
+#pragma unroll
+    for (int w = 0; w < 8; ++w) b[w] = bias ? bias[c + w] : 0.f;
+    uint4 past[K > 1 ? K - 1 : 1];       // past[j]: the input K - 1 - j tokens before this one
+    int row = -2;
+    const int n0 = blockIdx.y * CONV_RUN, n1 = min(n0 + CONV_RUN, n_tokens);
+    for (int n = n0; n < n1; ++n) {
+        const int r = token_row[n];
+        uint4 packed = make_uint4(0u, 0u, 0u, 0u);
+        if (r >= 0) {
+            if (r != row) {
+                const int i = n - row_start[r];
+                const bf16* st = state + (int64_t)row_slot[r] * (K - 1) * C;
+#pragma unroll
+                for (int j = 0; j < K - 1; ++j) {
+                    const int back = K - 1 - j;
+                    past[j] = *reinterpret_cast<const uint4*>(
+                        back <= i ? x + (int64_t)(n - back) * ldx + c : st + (int64_t)(i + j) * C + c);
+                }
+            }
+            const uint4 now = *reinterpret_cast<const uint4*>(x + (int64_t)n * ldx + c);
+            float acc[8];
+#pragma unroll
+            for (int w = 0; w < 8; ++w) acc[w] = b[w];
+#pragma unroll
+            for (int j = 0; j < K; ++j) {
+                const uint4 raw = j < K - 1 ? past[j] : now;
+                const bf16* e = reinterpret_cast<const bf16*>(&raw);
+#pragma unroll
+                for (int w = 0; w < 8; ++w) acc[w] = fmaf(tp[j][w], __bfloat162float(e[w]), acc[w]);
+            }
+            bf16* o = reinterpret_cast<bf16*>(&packed);
+#pragma unroll
+            for (int w = 0; w < 8; ++w) o[w] = __float2bfloat16_rn(acc[w] / (1.0f + expf(-acc[w])));
+#pragma unroll
+            for (int j = 0; j + 1 < K - 1; ++j) past[j] = past[j + 1];
+            if (K > 1) past[K > 1 ? K - 2 : 0] = now;
+        }
+        row = r;
+        *reinterpret_cast<uint4*>(out + (int64_t)n * C + c) = packed;
+    }
+}
+
 // state[slot, s, c] for s = 0 .. K-2 becomes entry n_new + s of (old state, the row's new inputs).
 // grid (ceil(C / 256), rows); rows without tokens are left alone.
 template <typename T>
@@ -161,7 +226,8 @@ __global__ void conv_state_update_kernel(const T* __restrict__ x, int64_t ldx, i
     }
 }
 
-// grid (tokens, ceil(H / 4)); one warp per (token, head).  o: [n_tokens, H * V] float;
+// grid (tokens, ceil(H / 4)); one warp per (token, head), or with `wide` (long heads) grid (tokens,
+// H) and all four warps on one head.  o: [n_tokens, H * V] float;
 // gate: rows ldg apart; out: rows ldo apart (a column slice of a wider buffer, or H * V).  gain has V entries (every head the same) or,
 // with gain_per_head, H * V.  gate_act: 0 = silu(gate), 1 = sigmoid(gate).  den / floor (may be
 // null): [n_tokens, H]; a head's o is first divided by max(|den|, floor) + 1e-6.
@@ -171,26 +237,28 @@ __global__ void __launch_bounds__(128)
 head_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ gate, int64_t ldg,
                       const float* __restrict__ gain, float eps, const float* __restrict__ den,
                       const float* __restrict__ floor, T* __restrict__ out, int64_t ldo, int H,
-                      int V, int gain_per_head, int gate_act) {
+                      int V, int gain_per_head, int gate_act, int wide) {
     pdl_wait();
     pdl_trigger();
+    __shared__ float scratch[33];
     const int64_t n = blockIdx.x;
-    const int head = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (head >= H) return;
+    const int head = wide ? blockIdx.y : blockIdx.y * 4 + (threadIdx.x >> 5);
+    const int lane = wide ? threadIdx.x : threadIdx.x & 31, lanes = wide ? 128 : 32;
+    if (head >= H) return;                             // (never with wide)
     const float* src = o + (n * H + head) * V;
     float by = 1.f;
     if (den) by = 1.0f / (fmaxf(fabsf(den[n * H + head]), floor[n * H + head]) + DIVISOR_FLOOR);
     float ss = 0.f;
-    for (int j = lane; j < V; j += 32) {
+    for (int j = lane; j < V; j += lanes) {
         const float v = src[j] * by;
         ss += v * v;
     }
-    ss = warp_sum(ss);
+    ss = wide ? block_sum(ss, scratch) : warp_sum(ss);
     const float inv = by / sqrtf(ss / (float)V + eps);
     const T* g = gate + n * ldg + (int64_t)head * V;
     const float* gn = gain + (gain_per_head ? (int64_t)head * V : 0);
     T* dst = out + n * ldo + (int64_t)head * V;
-    for (int j = lane; j < V; j += 32) {
+    for (int j = lane; j < V; j += lanes) {
         const float z = to_float(g[j]);
         const float sig = 1.0f / (1.0f + expf(-z));
         dst[j] = from_float<T>(src[j] * inv * gn[j] * (gate_act == 1 ? sig : z * sig));
@@ -471,6 +539,15 @@ SLLM_EXPORT int sllm_conv_silu(const void* x, int64_t ldx, const float* taps,
     if (C <= 0 || K < 1 || K > CONV_MAX_TAPS || ldx < C) return (int)cudaErrorInvalidValue;
     if (dtype == 1 && taps_t != nullptr && C % 8 == 0 && ldx % 8 == 0 &&
         !(((uintptr_t)x | (uintptr_t)state | (uintptr_t)out | (uintptr_t)taps_t) & 15)) {
+        if (n_tokens >= 256 && K <= 4 && (n_tokens + CONV_RUN - 1) / CONV_RUN <= 65535) {
+            dim3 grid((C / 8 + 127) / 128, (n_tokens + CONV_RUN - 1) / CONV_RUN);
+            typedef __nv_bfloat16 bf16;
+            auto run = K == 1 ? conv_silu_run_kernel<1> : K == 2 ? conv_silu_run_kernel<2>
+                     : K == 3 ? conv_silu_run_kernel<3> : conv_silu_run_kernel<4>;
+            return (int)sllm_launch_pdl(run, grid, dim3(128), 0, stream, (const bf16*)x, ldx, taps_t,
+                                        bias, (const bf16*)state, token_row, row_start, row_slot,
+                                        (bf16*)out, C, n_tokens);
+        }
         int64_t vblocks = ((int64_t)n_tokens * (C / 8) + 255) / 256;
         if (vblocks > 148 * 32) vblocks = 148 * 32;
         conv_silu_vec_kernel<<<(int)vblocks, 256, 0, stream>>>(
@@ -521,15 +598,17 @@ SLLM_EXPORT int sllm_head_norm_gate(const float* o, const void* gate, int64_t ld
     if (H <= 0 || V <= 0 || gate_act < 0 || gate_act > 1 || ldo < (int64_t)H * V ||
         (den == nullptr) != (floor == nullptr))
         return (int)cudaErrorInvalidValue;
-    dim3 grid(n_tokens, (H + 3) / 4);
+    const int wide = V >= 256;
+    dim3 grid(n_tokens, wide ? H : (H + 3) / 4);
+    if (H > 65535) return (int)cudaErrorInvalidValue;
     if (dtype == 0)
         head_norm_gate_kernel<float><<<grid, 128, 0, stream>>>(o, (const float*)gate, ldg, gain,
                                                                eps, den, floor, (float*)out, ldo, H, V,
-                                                               gain_per_head, gate_act);
+                                                               gain_per_head, gate_act, wide);
     else if (dtype == 1)
         head_norm_gate_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>(
             o, (const __nv_bfloat16*)gate, ldg, gain, eps, den, floor, (__nv_bfloat16*)out, ldo, H, V,
-            gain_per_head, gate_act);
+            gain_per_head, gate_act, wide);
     else
         return (int)cudaErrorInvalidValue;
     SLLM_LAUNCH_CHECK();

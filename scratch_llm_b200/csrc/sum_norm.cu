@@ -138,7 +138,8 @@ __global__ void __launch_bounds__(512) sum_norm_kernel(const SumNorm a) {
 // token is in last[slot], where the row's last token is left for the next step (by the block of
 // the row's first token, after it has read the old one).  ids as in embed_kernel (-1 - j stands
 // for pending[j]).  Padding tokens (token_row -1) take row `buckets`.  One block per token.
-template <typename T>
+// V: elements per access (4 where d allows it, else 1).
+template <typename T, int V>
 __global__ void embed_pair_kernel(const int* __restrict__ ids, const int* __restrict__ pending,
                                   const int* __restrict__ positions,
                                   const int* __restrict__ token_row,
@@ -175,8 +176,13 @@ __global__ void embed_pair_kernel(const int* __restrict__ ids, const int* __rest
     const T* a = table + (int64_t)id * d;
     const T* b = pairs + pair * d;
     float* dst = out + (int64_t)n * d;
-    for (int i = threadIdx.x; i < d; i += blockDim.x)
-        dst[i] = fmaf(to_float(a[i]), scale, to_float(b[i]));
+    for (int i = threadIdx.x * V; i < d; i += blockDim.x * V) {
+        const Few<V> x = few<V>(a + i), y = few<V>(b + i);
+        Few<V> z;
+#pragma unroll
+        for (int k = 0; k < V; ++k) z.v[k] = fmaf(x.v[k], scale, y.v[k]);
+        put<V>(dst + i, z);
+    }
 }
 
 }  // namespace sllm
@@ -240,16 +246,17 @@ SLLM_EXPORT int sllm_embed_pair(const int* ids, const int* pending, const int* p
                                 int n_tokens, int d, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (d <= 0 || buckets < 1 || mul_prev < 0 || mul_cur < 0) return (int)cudaErrorInvalidValue;
-    const int threads = d >= 256 ? 256 : 64;
-    if (dtype == 0)
-        return (int)sllm_launch_pdl(embed_pair_kernel<float>, dim3(n_tokens), dim3(threads), 0, stream,
-                                    ids, pending, positions, token_row, row_start, row_slot,
-                                    (const float*)table, (const float*)pairs, last, mul_prev, mul_cur,
-                                    buckets, scale, out, d);
-    if (dtype == 1)
-        return (int)sllm_launch_pdl(embed_pair_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0,
-                                    stream, ids, pending, positions, token_row, row_start, row_slot,
-                                    (const __nv_bfloat16*)table, (const __nv_bfloat16*)pairs, last,
-                                    mul_prev, mul_cur, buckets, scale, out, d);
+    const int threads = d >= 1024 ? 256 : 64;
+    const bool vec = d % 4 == 0 && !(((uintptr_t)table | (uintptr_t)pairs | (uintptr_t)out) & 15);
+#define SLLM_EP(T, V)                                                                              \
+    return (int)sllm_launch_pdl(embed_pair_kernel<T, V>, dim3(n_tokens), dim3(threads), 0, stream, \
+                                ids, pending, positions, token_row, row_start, row_slot,          \
+                                (const T*)table, (const T*)pairs, last, mul_prev, mul_cur,        \
+                                buckets, scale, out, d)
+    if (dtype == 0 && vec) SLLM_EP(float, 4);
+    if (dtype == 0) SLLM_EP(float, 1);
+    if (dtype == 1 && vec) SLLM_EP(__nv_bfloat16, 4);
+    if (dtype == 1) SLLM_EP(__nv_bfloat16, 1);
+#undef SLLM_EP
     return (int)cudaErrorInvalidValue;
 }

@@ -110,6 +110,7 @@ class StepBatch:
     n_single: int = 0
     n_multi: int = 0
     max_new_multi: int = 0
+    min_new: int = 1          # the fewest tokens a row brings (a lower bound)
     max_context_single: int = 0
     context_bucket: int = 0   # max_context_single rounded up to a power of two (at least 256)
     #: the logits of every token are wanted, in the tokens' order (a decode step: the gather of
@@ -296,7 +297,7 @@ def build_batch(cache, stager: BatchStager, rows: Sequence[RowInput], vocab_size
         token_ids=dev[0], positions=dev[1], token_row=dev[2], row_start=dev[3],
         row_pos0=dev[4], row_slot=dev[5], logit_index=dev[6], single_rows=dev[7],
         multi_rows=dev[8], block_tables=dev[9:], n_single=len(single), n_multi=len(multi),
-        max_new_multi=max((lens[i] for i in multi), default=0),
+        max_new_multi=max((lens[i] for i in multi), default=0), min_new=min(lens),
         max_context_single=ctx_single, context_bucket=context_bucket(ctx_single),
         wants_every_token=bool(li.size == n_tokens and (li == np.arange(n_tokens)).all()),
         host_row_new=lens, host_row_pos0=row_pos0.tolist(), n_real_tokens=n_tokens,

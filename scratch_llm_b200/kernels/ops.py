@@ -2058,7 +2058,7 @@ def embed_pair(ids: torch.Tensor, positions: torch.Tensor, token_row: torch.Tens
 #: the scan takes key sizes up to this
 GATED_SCAN_MAX_KEY_DIM = 1024
 #: rows of at least this many tokens take the chunk kernels where these take the sizes
-GATED_SCAN_MIN_CHUNKED = 32
+GATED_SCAN_MIN_CHUNKED = 64
 
 
 def gated_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: torch.Tensor,
@@ -2066,7 +2066,7 @@ def gated_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: tor
                row_slot: torch.Tensor, out: torch.Tensor, n_rows: int, n_groups: int, key_dim: int,
                value_dim: int, longest: int, ones_out: torch.Tensor | None = None,
                skip: torch.Tensor | None = None, scale: float = 1.0,
-               min_chunked: int | None = None) -> torch.Tensor:
+               min_chunked: int | None = None, shortest: int = 1) -> torch.Tensor:
     """The recurrence ``S <- exp(log_decay) S + weight k v^T``, ``out = scale S^T q + skip v`` over
     the packed batch (csrc/gated_scan.cu): ``q``, ``k`` [N, G * key_dim] and ``v`` [N, H *
     value_dim] (may be column slices; head h reads group ``h // (H / G)``), ``log_decay`` (at
@@ -2075,7 +2075,8 @@ def gated_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: tor
     it is [slots, H, value_dim + 1, key_dim] and its last column belongs to a value that is
     always 1 (a normaliser), whose read-out (times ``scale``) goes there.  ``longest``: the most
     tokens a row brings (an upper bound).  ``min_chunked``: rows of at least so many tokens run in
-    chunks on the tensor cores (bfloat16, sizes in multiples of 16 and 8; 0: never)."""
+    chunks on the tensor cores (bfloat16, sizes in multiples of 16 and 8; 0: never).
+    ``shortest``: the fewest tokens a row brings (a lower bound)."""
     _need(q, None, "q", contiguous=False)
     _need(k, q.dtype, "k", contiguous=False)
     _need(v, q.dtype, "v", contiguous=False)
@@ -2119,7 +2120,8 @@ def gated_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: tor
         c_int64(v.stride(0)), _ptr(log_decay), _ptr(weight), _ptr(state), _ptr(row_start),
         _ptr(row_slot), _ptr(out), _ptr(ones_out), _ptr(skip), c_float(scale), c_int(n),
         c_int(n_rows), c_int(n_heads), c_int(n_groups), c_int(key_dim), c_int(value_dim),
-        c_int(ones), c_int(int(chunked)), c_int(min_chunked), c_int(longest), _ptr(dS),
+        c_int(ones), c_int(int(chunked)), c_int(min_chunked), c_int(shortest), c_int(longest),
+        _ptr(dS),
         _ptr(decay), c_int(_code(q.dtype)), _stream()),
         "gated_scan_chunked" if chunked else "gated_scan")
     return out

@@ -109,6 +109,7 @@ class MatrixMemory(Mixer):
         o = make((n, H * V), dtype=torch.float32, device=proj.device)
         ops.gated_scan(q, k, v, log_decay, weight, S, batch.row_start, batch.row_slot, o,
                        batch.n_rows, H, D, V, longest=1 if one_each else batch.max_new,
+                       shortest=batch.min_new,
                        ones_out=den, scale=D ** -0.5)
         out = torch.empty((n, H * V), dtype=proj.dtype, device=proj.device)
         ops.head_norm_gate(o, g, self.gain, self.eps, out, H, gate_activation="sigmoid",

@@ -124,6 +124,9 @@ class RoutedExperts(FeedForward):
         router = [put(tensors["router"])]
         if self.shared_gate:      # one more output of the router's product
             router.append(put(tensors["shared.sg"]))
+        # (zero rows up to a multiple of 8: the library's products are slow for odd widths)
+        rows = sum(t.shape[0] for t in router)
+        router.append(router[0].new_zeros((-rows % 8, self.hidden_size)))
         self.router = Linear(torch.cat(router, 0).contiguous())
         if self.has_correction:
             self.correction = tensors["correction"].to(device=ctx.device,
@@ -146,10 +149,9 @@ class RoutedExperts(FeedForward):
     def forward(self, x, lazy: bool = False):
         n, d = x.shape
         logits = self.router(x, out_dtype=torch.float32)
-        gate = None
-        if self.shared_gate:
-            total = self.experts + self.identity
-            logits, gate = logits[:, :total], logits[:, total:]
+        total = self.experts + self.identity
+        gate = logits[:, total:total + 1] if self.shared_gate else None
+        logits = logits[:, :total]
         tensor_cores = self._tensor_cores(x.dtype)
         ids, weights, pair_token, pair_place, meta, max_tiles, rows = ops.moe_route(
             logits, self.correction, None, self.experts, self.groups, self.keep_groups, self.top,

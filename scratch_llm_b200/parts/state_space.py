@@ -126,7 +126,8 @@ class StateSpace(Mixer):
         ops.gated_scan(act[:, self.inner + G * N:], act[:, self.inner:self.inner + G * N],
                        act[:, :self.inner], gates[0], gates[1], S, batch.row_start,
                        batch.row_slot, y, batch.n_rows, G, N, V,
-                       longest=batch.max_new if batch.n_multi else 1, skip=self.skip)
+                       longest=batch.max_new if batch.n_multi else 1,
+                       shortest=batch.min_new, skip=self.skip)
         out = torch.empty((n, self.inner), dtype=proj.dtype, device=proj.device)
         ops.gate_part_norm(y, proj[:, self.z_col:self.z_col + self.inner], self.gain, self.eps,
                            self.norm_groups, out)
