@@ -102,6 +102,34 @@ __global__ void __launch_bounds__(256) gated_scan_kernel(const ScanArgs a, int t
             for (int w = 0; w < 4; ++w) S[4 * i + w] = (live && e + w < N) ? st[e + w] : 0.f;
         }
     }
+    if (n_new == 1 && quads && a.vec4) {       // decoding: nothing is staged
+        const int64_t n = t0;
+        const float decay = expf(a.log_a[n * H + head]);
+        const float value = !is_ones ? to_float(v[n * a.ldv + col]) : 1.f;
+        const float bv = a.b[n * H + head] * value;
+        float acc = 0.f;
+#pragma unroll
+        for (int i = 0; i < QPL; ++i) {
+            const int e = (i * LPC + sub) * 4;
+            if (e < N) {
+                const float4 kk = load4(k + n * a.ldk + e), qq = load4(q + n * a.ldq + e);
+                float4 x;
+                x.x = fmaf(decay, S[4 * i], bv * kk.x);
+                x.y = fmaf(decay, S[4 * i + 1], bv * kk.y);
+                x.z = fmaf(decay, S[4 * i + 2], bv * kk.z);
+                x.w = fmaf(decay, S[4 * i + 3], bv * kk.w);
+                acc = fmaf(x.x, qq.x, fmaf(x.y, qq.y, fmaf(x.z, qq.z, fmaf(x.w, qq.w, acc))));
+                if (live) *reinterpret_cast<float4*>(st + e) = x;
+            }
+        }
+#pragma unroll
+        for (int o = LPC / 2; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+        if (sub == 0 && live) {
+            if (is_ones) a.ones_out[n * H + head] = acc * a.scale;
+            else a.out[n * H * V + (int64_t)head * V + col] = fmaf(skip, value, acc * a.scale);
+        }
+        return;
+    }
     const int NP = (N + 3) / 4 * 4;            // staged rows, padded with zeros
     float* ks = sm;                            // [tokens_staged][NP]
     float* qs = ks + tokens_staged * NP;       // [tokens_staged][NP]

@@ -22,6 +22,13 @@ namespace sllm {
 
 constexpr int CONV_MAX_TAPS = 16;
 
+// sigmoid(z): exact rounding steps on the 32-bit path; where the result is rounded to bfloat16 the
+// hardware's exponential and division (relative error around 1e-6).
+template <typename T> __device__ __forceinline__ float sigmoid_of(float z) {
+    if (sizeof(T) == 4) return 1.0f / (1.0f + expf(-z));
+    return __fdividef(1.0f, 1.0f + __expf(-z));
+}
+
 // V consecutive values (4: 16 or 8 bytes at a time, suitably aligned; 1: one by one).
 template <int V> __device__ __forceinline__ void load_few(const float* p, float* v) {
     if (V == 4) {
@@ -88,7 +95,7 @@ __global__ void conv_silu_kernel(const T* __restrict__ x, int64_t ldx,
             else v = to_float(st[(int64_t)(i + j) * C + c]);   // i - back + (K - 1)
             acc = fmaf(taps[(int64_t)c * K + j], v, acc);
         }
-        out[idx] = from_float<T>(acc / (1.0f + expf(-acc)));
+        out[idx] = from_float<T>(acc * sigmoid_of<T>(acc));
     }
 }
 
@@ -134,7 +141,7 @@ __global__ void conv_silu_vec_kernel(const __nv_bfloat16* __restrict__ x, int64_
             }
             bf16* o = reinterpret_cast<bf16*>(&packed);
 #pragma unroll
-            for (int w = 0; w < 8; ++w) o[w] = __float2bfloat16_rn(acc[w] / (1.0f + expf(-acc[w])));
+            for (int w = 0; w < 8; ++w) o[w] = __float2bfloat16_rn(acc[w] * sigmoid_of<bf16>(acc[w]));
         }
         *reinterpret_cast<uint4*>(out + n * C + c) = packed;
     }
@@ -165,11 +172,22 @@ conv_silu_run_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx,
     }
 #pragma unroll
     for (int w = 0; w < 8; ++w) b[w] = bias ? bias[c + w] : 0.f;
+    const int n0 = blockIdx.y * CONV_RUN;
+    int rows[CONV_RUN];                  // -1: padding, or beyond the last token
+    uint4 in[CONV_RUN];                  // every input of the run is requested at once
+#pragma unroll
+    for (int i = 0; i < CONV_RUN; ++i) {
+        const bool there = n0 + i < n_tokens;
+        rows[i] = there ? token_row[n0 + i] : -1;
+        in[i] = there ? *reinterpret_cast<const uint4*>(x + (int64_t)(n0 + i) * ldx + c)
+                      : make_uint4(0u, 0u, 0u, 0u);
+    }
     uint4 past[K > 1 ? K - 1 : 1];       // past[j]: the input K - 1 - j tokens before this one
     int row = -2;
-    const int n0 = blockIdx.y * CONV_RUN, n1 = min(n0 + CONV_RUN, n_tokens);
-    for (int n = n0; n < n1; ++n) {
-        const int r = token_row[n];
+#pragma unroll
+    for (int k = 0; k < CONV_RUN; ++k) {
+        const int n = n0 + k, r = rows[k];
+        if (n >= n_tokens) break;
         uint4 packed = make_uint4(0u, 0u, 0u, 0u);
         if (r >= 0) {
             if (r != row) {
@@ -182,7 +200,7 @@ conv_silu_run_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx,
                         back <= i ? x + (int64_t)(n - back) * ldx + c : st + (int64_t)(i + j) * C + c);
                 }
             }
-            const uint4 now = *reinterpret_cast<const uint4*>(x + (int64_t)n * ldx + c);
+            const uint4 now = in[k];
             float acc[8];
 #pragma unroll
             for (int w = 0; w < 8; ++w) acc[w] = b[w];
@@ -195,7 +213,7 @@ conv_silu_run_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx,
             }
             bf16* o = reinterpret_cast<bf16*>(&packed);
 #pragma unroll
-            for (int w = 0; w < 8; ++w) o[w] = __float2bfloat16_rn(acc[w] / (1.0f + expf(-acc[w])));
+            for (int w = 0; w < 8; ++w) o[w] = __float2bfloat16_rn(acc[w] * sigmoid_of<bf16>(acc[w]));
 #pragma unroll
             for (int j = 0; j + 1 < K - 1; ++j) past[j] = past[j + 1];
             if (K > 1) past[K > 1 ? K - 2 : 0] = now;
@@ -226,25 +244,26 @@ __global__ void conv_state_update_kernel(const T* __restrict__ x, int64_t ldx, i
     }
 }
 
-// grid (tokens, ceil(H / 4)); one warp per (token, head), or with `wide` (long heads) grid (tokens,
+// grid (tokens, ceil(H / 4)); one warp per (token, head), or with WIDE (long heads) grid (tokens,
 // H) and all four warps on one head.  o: [n_tokens, H * V] float;
 // gate: rows ldg apart; out: rows ldo apart (a column slice of a wider buffer, or H * V).  gain has V entries (every head the same) or,
 // with gain_per_head, H * V.  gate_act: 0 = silu(gate), 1 = sigmoid(gate).  den / floor (may be
 // null): [n_tokens, H]; a head's o is first divided by max(|den|, floor) + 1e-6.
 constexpr float DIVISOR_FLOOR = 1e-6f;
-template <typename T>
+template <typename T, bool WIDE>
 __global__ void __launch_bounds__(128)
 head_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ gate, int64_t ldg,
                       const float* __restrict__ gain, float eps, const float* __restrict__ den,
                       const float* __restrict__ floor, T* __restrict__ out, int64_t ldo, int H,
-                      int V, int gain_per_head, int gate_act, int wide) {
+                      int V, int gain_per_head, int gate_act) {
     pdl_wait();
     pdl_trigger();
     __shared__ float scratch[33];
     const int64_t n = blockIdx.x;
-    const int head = wide ? blockIdx.y : blockIdx.y * 4 + (threadIdx.x >> 5);
-    const int lane = wide ? threadIdx.x : threadIdx.x & 31, lanes = wide ? 128 : 32;
-    if (head >= H) return;                             // (never with wide)
+    const int head = WIDE ? blockIdx.y : blockIdx.y * 4 + (threadIdx.x >> 5);
+    const int lane = WIDE ? threadIdx.x : threadIdx.x & 31;
+    constexpr int lanes = WIDE ? 128 : 32;
+    if (head >= H) return;                             // (never with WIDE)
     const float* src = o + (n * H + head) * V;
     float by = 1.f;
     if (den) by = 1.0f / (fmaxf(fabsf(den[n * H + head]), floor[n * H + head]) + DIVISOR_FLOOR);
@@ -253,14 +272,14 @@ head_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ gate, i
         const float v = src[j] * by;
         ss += v * v;
     }
-    ss = wide ? block_sum(ss, scratch) : warp_sum(ss);
+    ss = WIDE ? block_sum(ss, scratch) : warp_sum(ss);
     const float inv = by / sqrtf(ss / (float)V + eps);
     const T* g = gate + n * ldg + (int64_t)head * V;
     const float* gn = gain + (gain_per_head ? (int64_t)head * V : 0);
     T* dst = out + n * ldo + (int64_t)head * V;
     for (int j = lane; j < V; j += lanes) {
         const float z = to_float(g[j]);
-        const float sig = 1.0f / (1.0f + expf(-z));
+        const float sig = sigmoid_of<T>(z);
         dst[j] = from_float<T>(src[j] * inv * gn[j] * (gate_act == 1 ? sig : z * sig));
     }
 }
@@ -410,7 +429,7 @@ gate_part_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, i
         load_few<V>(gate + n * ldg + at + i, z);
 #pragma unroll
         for (int k = 0; k < V; ++k) {
-            v[k] *= z[k] / (1.0f + expf(-z[k]));
+            v[k] *= z[k] * sigmoid_of<T>(z[k]);
             ss = fmaf(v[k], v[k], ss);
             gp_row[i + k] = v[k];
         }
@@ -598,19 +617,20 @@ SLLM_EXPORT int sllm_head_norm_gate(const float* o, const void* gate, int64_t ld
     if (H <= 0 || V <= 0 || gate_act < 0 || gate_act > 1 || ldo < (int64_t)H * V ||
         (den == nullptr) != (floor == nullptr))
         return (int)cudaErrorInvalidValue;
-    const int wide = V >= 256;
+    const int wide = V >= 256 && (int64_t)n_tokens * H <= 1024;
     dim3 grid(n_tokens, wide ? H : (H + 3) / 4);
     if (H > 65535) return (int)cudaErrorInvalidValue;
-    if (dtype == 0)
-        head_norm_gate_kernel<float><<<grid, 128, 0, stream>>>(o, (const float*)gate, ldg, gain,
-                                                               eps, den, floor, (float*)out, ldo, H, V,
-                                                               gain_per_head, gate_act, wide);
-    else if (dtype == 1)
-        head_norm_gate_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>(
-            o, (const __nv_bfloat16*)gate, ldg, gain, eps, den, floor, (__nv_bfloat16*)out, ldo, H, V,
-            gain_per_head, gate_act, wide);
-    else
-        return (int)cudaErrorInvalidValue;
+    typedef __nv_bfloat16 bf16;
+#define SLLM_HNG(T, WIDE)                                                                          \
+    head_norm_gate_kernel<T, WIDE><<<grid, 128, 0, stream>>>(o, (const T*)gate, ldg, gain, eps, den, \
+                                                             floor, (T*)out, ldo, H, V,            \
+                                                             gain_per_head, gate_act)
+    if (dtype == 0 && wide) SLLM_HNG(float, true);
+    else if (dtype == 0) SLLM_HNG(float, false);
+    else if (dtype == 1 && wide) SLLM_HNG(bf16, true);
+    else if (dtype == 1) SLLM_HNG(bf16, false);
+    else return (int)cudaErrorInvalidValue;
+#undef SLLM_HNG
     SLLM_LAUNCH_CHECK();
     return 0;
 }
