@@ -256,8 +256,8 @@ def engine_of(cfg, capacity_tokens: int, max_requests: int, page_size: int):
 
 
 def compare_main(args) -> int:
-    """--compare nilevik | vobosun | titedra | tubevik | deganex: prefill and decode throughput of that design beside
-    the engine's other models of equal size (for Vobosun: Nilevik, the closest one, a hybrid of
+    """--compare nilevik | vobosun | titedra | tubevik | deganex: prefill and decode throughput of
+    that design beside the engine's other models of equal size (for Vobosun: Nilevik, the closest one, a hybrid of
     attention and a delta rule with normed branch outputs, and the Llama-style model; for
     Titedra: Vobosun, the closest one, with norms around every branch, a partly rotated
     attention and routed experts, and the Llama-style model; for Tubevik: Nilevik, the closest one, likewise a hybrid of windowed

@@ -1402,7 +1402,8 @@ def moe_route(logits: torch.Tensor, correction: torch.Tensor | None, token_row: 
               gather_from: torch.Tensor | None = None, flags: int = 0):
     """Route every token of ``logits`` (float32 [N, outputs], may be a column slice) and sort the
     (token, choice) pairs by expert (csrc/moe.cu).  Returns ``(ids [N, top], weights [N, top],
-    pair_token [N * top], pair_place [N * top], meta, max_tiles, rows)``; ``meta`` is the tile list of the grouped
+    pair_token [N * top], pair_place [N * top], meta, max_tiles, rows)``; ``meta`` is the tile list
+    of the grouped
     products, in tiles of ``tile_rows`` rows (default: what :func:`moe_product` takes).
     ``gather_from`` (bfloat16 [N, K], K % 8 == 0): the caller wants the tokens' rows in the
     sorted order; ``rows`` is that copy where the router made it on its way (steps of few tokens,
@@ -1816,9 +1817,9 @@ def latent_small(x: torch.Tensor, x_head_stride: int, w: torch.Tensor, out: torc
     ``out[n, h * out_head_stride + j] = f * sum_k x[n, h * x_head_stride + k] * w[h, k, j]`` for
     ``w`` [H, K, J] (the output index last).  ``gate`` [N, H] (may be a column slice): ``f =
     sigmoid(gate[n, h])``; [N, H * J]: ``f = sigmoid(gate[n, h * J + j])``.  ``rot = (rot_dim,
-    positions, cos, sin)``: the head's next ``rot_dim`` entries of ``x`` go behind the J outputs, the first ``2 * cos.shape[1]`` of them rotated by
-    the token's position (as :func:`latent_q_rot` does), zeros behind them up to
-    ``out_head_stride``."""
+    positions, cos, sin)``: the head's next ``rot_dim`` entries of ``x`` go behind the J outputs, the
+    first ``2 * cos.shape[1]`` of them rotated by the token's position (as :func:`latent_q_rot`
+    does), zeros behind them up to ``out_head_stride``."""
     _need(x, None, "x", contiguous=False)
     _need(w, x.dtype, "w")
     _need(out, x.dtype, "out", contiguous=False)

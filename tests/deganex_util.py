@@ -52,9 +52,9 @@ def _with_again(layers, *which):
 
 
 # Sizes differ from one configuration to the next in everything: each kind of mixer first, layers
-# that run once and twice, head counts from 1 to 6, value sizes smaller and larger
-# than key sizes and beyond 64, groups of 1 and of every head, one to four convolution taps, one
-# norm part and as many as do not line up with the heads, cached vectors that are and are not a
+# that run once and twice, head counts from 1 to 6, value sizes smaller and larger than key sizes
+# and beyond 64, groups of 1 and of every head, one to four convolution taps, one norm part and as
+# many as do not line up with the heads, cached vectors that are and are not a
 # multiple of 16 (and of 64), layers without a feed-forward, without a shared expert, one choice
 # and all of them, tables of one and of many buckets, multipliers of 0 and larger than the table,
 # with and without caps.
