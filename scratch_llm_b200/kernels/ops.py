@@ -1403,8 +1403,7 @@ def moe_route(logits: torch.Tensor, correction: torch.Tensor | None, token_row: 
     """Route every token of ``logits`` (float32 [N, outputs], may be a column slice) and sort the
     (token, choice) pairs by expert (csrc/moe.cu).  Returns ``(ids [N, top], weights [N, top],
     pair_token [N * top], pair_place [N * top], meta, max_tiles, rows)``; ``meta`` is the tile list
-    of the grouped
-    products, in tiles of ``tile_rows`` rows (default: what :func:`moe_product` takes).
+    of the grouped products, in tiles of ``tile_rows`` rows (default: what :func:`moe_product` takes).
     ``gather_from`` (bfloat16 [N, K], K % 8 == 0): the caller wants the tokens' rows in the
     sorted order; ``rows`` is that copy where the router made it on its way (steps of few tokens,
     where one CTA does everything in one launch), else None (:func:`moe_gather_rows` makes it).

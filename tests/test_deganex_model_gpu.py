@@ -230,7 +230,7 @@ def test_greedy_generation_through_the_scheduler(name, models):
     gives the plain model's greedy continuation."""
     from scratch_llm_b200 import LLM, SamplingParams
     cfg, tensors, folder, reqs, _ = models[name]
-    prompts = [toks for toks in reqs.values() if len(toks) >= 2][:5]
+    prompts = [toks for toks in reqs.values() if 2 <= len(toks) <= 100][:5]
     n_new = 12
 
     def plain_greedy(prompt):
