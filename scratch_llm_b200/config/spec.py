@@ -110,8 +110,14 @@ class ModelSpec:
     #: sizes), with its tensor-name prefix; None: the tokens' vectors alone
     token_embedding: PartSpec | None = None
     token_embedding_name: str = ""
+    #: the residual stream has this many parts, all equal to the embedding output at the start; the
+    #: blocks say how sublayers read and write them, and the final norm reads their sum.  None: one
+    #: sum, as usual
+    streams: int | None = None
 
     def __post_init__(self) -> None:
+        if self.streams is not None and self.streams < 1:
+            raise ValueError(f"streams must be at least 1, got {self.streams}")
         if self.position_sinusoid_base < 0:
             raise ValueError("position_sinusoid_base must not be negative")
         if self.logit_softcap < 0:

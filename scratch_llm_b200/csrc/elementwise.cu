@@ -8,20 +8,24 @@
 
 namespace sllm {
 
-// out[n, :] = table[ids[n], :] as float, times scale.  One block per token.  An id -1 - j stands
+// out[n, s, :] = table[ids[n], :] as float, times scale, for s = 0 .. copies - 1 (a residual stream
+// of several equal parts at its start; else copies is 1).  One block per token.  An id -1 - j stands
 // for pending[j]: a token that an earlier kernel of the stream chose and the host has not read yet.
 template <typename T>
 __global__ void embed_kernel(const int* __restrict__ ids, const int* __restrict__ pending,
                              const T* __restrict__ table, float* __restrict__ out, int d,
-                             float scale) {
+                             float scale, int copies) {
     pdl_wait();
     pdl_trigger();
     const int64_t n = blockIdx.x;
     int id = ids[n];
     if (id < 0) id = pending[-1 - id];
     const T* src = table + (int64_t)id * d;
-    float* dst = out + n * d;
-    for (int i = threadIdx.x; i < d; i += blockDim.x) dst[i] = to_float(src[i]) * scale;
+    float* dst = out + n * copies * d;
+    for (int i = threadIdx.x; i < d; i += blockDim.x) {
+        const float v = to_float(src[i]) * scale;
+        for (int s = 0; s < copies; ++s) dst[(int64_t)s * d + i] = v;
+    }
 }
 
 // The embedding with the first norm prepared for the product after it (up to 8 tokens, bfloat16
@@ -280,16 +284,17 @@ SLLM_EXPORT int sllm_logit_cap(float* x, int64_t n, float scale, float cap, cuda
 }
 
 SLLM_EXPORT int sllm_embed(const int* ids, const int* pending, const void* table, float* out,
-                           int n_tokens, int d, int dtype, float scale, cudaStream_t stream) {
+                           int n_tokens, int d, int dtype, float scale, int copies,
+                           cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (d <= 0) return (int)cudaErrorInvalidValue;
+    if (d <= 0 || copies < 1) return (int)cudaErrorInvalidValue;
     const int threads = norm_threads(d);
     if (dtype == 0)
         embed_kernel<float><<<n_tokens, threads, 0, stream>>>(ids, pending, (const float*)table, out,
-                                                              d, scale);
+                                                              d, scale, copies);
     else if (dtype == 1)
         embed_kernel<__nv_bfloat16><<<n_tokens, threads, 0, stream>>>(
-            ids, pending, (const __nv_bfloat16*)table, out, d, scale);
+            ids, pending, (const __nv_bfloat16*)table, out, d, scale, copies);
     else
         return (int)cudaErrorInvalidValue;
     SLLM_LAUNCH_CHECK();

@@ -7,7 +7,10 @@
 // state-space layer (SSD) is this with k = B, q = C, a = exp(-rate dt), b = dt and a skip; a
 // matrix memory with exponential gates is this with stabilised gates and a NORMALISER n <- a n +
 // b k, which is one more column of S whose value is always 1 (`ones`): its read-out q . n goes to
-// an array of its own.  The state is stored [slots, H, V (+ 1), N].
+// an array of its own.  Decays that are constants of the heads (lightning attention) are read from
+// one array for all tokens (ld_gates 0), with b = 1 (b null); q, k and v may come ahead of a silu,
+// which the first kernel then applies while it reads them.  The state is stored [slots, H, V (+ 1),
+// N].
 //
 // gated_scan_kernel (any sizes, both dtypes, all arithmetic 32-bit): columns of S are
 // independent.  LPC lanes share a column (EPL elements each, in quads), a CTA of 8 warps takes
@@ -29,11 +32,10 @@
 // is the state's way through memory, so they run as mma.sync from shared memory, without the
 // set-up of a TMEM accumulator.
 //
-// The chunk that starts at token t of the batch, in row r, has slot t / TC + r (distinct for
-// distinct chunks, whatever the rows' lengths), so a launch over slots finds its chunk on the
+// Chunks have slots (scan_chunks.cuh), so a launch over slots finds its chunk on the
 // device and nothing is read on the host.  Rows of fewer than `min_chunked` tokens are the first
 // kernel's, the others the chunk kernels'.
-#include "common.cuh"
+#include "scan_chunks.cuh"
 
 namespace sllm {
 
@@ -41,7 +43,8 @@ struct ScanArgs {
     const void* q; int64_t ldq;          // [tokens, >= G * N]
     const void* k; int64_t ldk;          // [tokens, >= G * N]
     const void* v; int64_t ldv;          // [tokens, >= H * V]
-    const float* log_a; const float* b;  // [tokens, H]
+    const float* log_a; const float* b;  // [tokens, H]; b null: 1
+    int64_t ld_gates;                    // H, or 0: log_a is [H] for all tokens
     float* state;                        // [slots, H, VX, N], VX = V + ones
     const int* row_start; const int* row_slot;
     float* out;                          // [tokens, H * V]
@@ -50,6 +53,7 @@ struct ScanArgs {
     float scale;
     int H, G, N, V, VX;
     int vec4;                            // rows of q and k allow reads of four elements
+    int silu;                            // token-by-token kernel: q, k and v pass a silu
     int min_chunked;                     // rows of at least so many tokens are the chunk kernels'
     // chunk kernels only
     float* dS;                           // [slots of chunks, H, VX, N]
@@ -57,11 +61,9 @@ struct ScanArgs {
     int n_rows;
 };
 
-__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
-    const uint2 raw = *reinterpret_cast<const uint2*>(p);
-    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
-    return make_float4(__low2float(h[0]), __high2float(h[0]), __low2float(h[1]), __high2float(h[1]));
+__device__ __forceinline__ float silu_if(float z, int on) { return on ? z / (1.0f + expf(-z)) : z; }
+__device__ __forceinline__ float4 silu_if(float4 z, int on) {
+    return on ? make_float4(silu_if(z.x, 1), silu_if(z.y, 1), silu_if(z.z, 1), silu_if(z.w, 1)) : z;
 }
 
 // ------------------------------------------------------------------------ token by token
@@ -104,15 +106,16 @@ __global__ void __launch_bounds__(256) gated_scan_kernel(const ScanArgs a, int t
     }
     if (n_new == 1 && quads && a.vec4) {       // decoding: nothing is staged
         const int64_t n = t0;
-        const float decay = expf(a.log_a[n * H + head]);
-        const float value = !is_ones ? to_float(v[n * a.ldv + col]) : 1.f;
-        const float bv = a.b[n * H + head] * value;
+        const float decay = expf(a.log_a[n * a.ld_gates + head]);
+        const float value = !is_ones ? silu_if(to_float(v[n * a.ldv + col]), a.silu) : 1.f;
+        const float bv = a.b ? a.b[n * H + head] * value : value;
         float acc = 0.f;
 #pragma unroll
         for (int i = 0; i < QPL; ++i) {
             const int e = (i * LPC + sub) * 4;
             if (e < N) {
-                const float4 kk = load4(k + n * a.ldk + e), qq = load4(q + n * a.ldq + e);
+                const float4 kk = silu_if(load4(k + n * a.ldk + e), a.silu);
+                const float4 qq = silu_if(load4(q + n * a.ldq + e), a.silu);
                 float4 x;
                 x.x = fmaf(decay, S[4 * i], bv * kk.x);
                 x.y = fmaf(decay, S[4 * i + 1], bv * kk.y);
@@ -145,24 +148,24 @@ __global__ void __launch_bounds__(256) gated_scan_kernel(const ScanArgs a, int t
             for (int i = tid; i < nt * per; i += 256) {
                 const int t = i / per, e = (i - t * per) * 4;
                 const int64_t n = t0 + c0 + t;
-                *reinterpret_cast<float4*>(ks + t * NP + e) = load4(k + n * a.ldk + e);
-                *reinterpret_cast<float4*>(qs + t * NP + e) = load4(q + n * a.ldq + e);
+                *reinterpret_cast<float4*>(ks + t * NP + e) = silu_if(load4(k + n * a.ldk + e), a.silu);
+                *reinterpret_cast<float4*>(qs + t * NP + e) = silu_if(load4(q + n * a.ldq + e), a.silu);
             }
         } else {
             for (int i = tid; i < nt * NP; i += 256) {
                 const int t = i / NP, e = i - t * NP;
                 const int64_t n = t0 + c0 + t;
-                ks[i] = e < N ? to_float(k[n * a.ldk + e]) : 0.f;
-                qs[i] = e < N ? to_float(q[n * a.ldq + e]) : 0.f;
+                ks[i] = e < N ? silu_if(to_float(k[n * a.ldk + e]), a.silu) : 0.f;
+                qs[i] = e < N ? silu_if(to_float(q[n * a.ldq + e]), a.silu) : 0.f;
             }
         }
         for (int i = tid; i < nt * COLS; i += 256) {
             const int t = i / COLS, j = col0 + i - t * COLS;
-            vs[i] = j < V ? to_float(v[(int64_t)(t0 + c0 + t) * a.ldv + j]) : 1.f;
+            vs[i] = j < V ? silu_if(to_float(v[(int64_t)(t0 + c0 + t) * a.ldv + j]), a.silu) : 1.f;
         }
         for (int t = tid; t < nt; t += 256) {
-            as[t] = expf(a.log_a[(int64_t)(t0 + c0 + t) * H + head]);
-            bs[t] = a.b[(int64_t)(t0 + c0 + t) * H + head];
+            as[t] = expf(a.log_a[(int64_t)(t0 + c0 + t) * a.ld_gates + head]);
+            bs[t] = a.b ? a.b[(int64_t)(t0 + c0 + t) * H + head] : 1.f;
         }
         __syncthreads();
         for (int t = 0; t < nt; ++t) {
@@ -212,7 +215,6 @@ __global__ void __launch_bounds__(256) gated_scan_kernel(const ScanArgs a, int t
 
 // --------------------------------------------------------------------------- chunk kernels
 
-constexpr int TC = 64;          // tokens of a chunk
 constexpr int VB = 64;          // columns of S per CTA (and the column of ones beside the last)
 constexpr int VT = VB + 8;      // columns staged
 constexpr int PARTS = 3;        // bfloat16 parts of a 32-bit operand
@@ -255,44 +257,18 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t* part) {
     }
 }
 
-// The row and the first token (within the row) of chunk slot `s`; false: no chunk has it.
-__device__ __forceinline__ bool find_chunk(const ScanArgs& a, int s, int& row, int& t0, int& c0,
-                                           int& n_new) {
-    const int lane = threadIdx.x & 31;
-    for (int r0 = 0; r0 < a.n_rows; r0 += 32) {
-        const int r = r0 + lane;
-        bool mine = false;
-        int start = 0, count = 0;
-        if (r < a.n_rows) {
-            start = a.row_start[r];
-            count = a.row_start[r + 1] - start;
-            const int first = start / TC + r;
-            mine = count >= a.min_chunked && s >= first && (s - first) * TC < count;
-        }
-        const unsigned hit = __ballot_sync(0xffffffffu, mine);
-        if (hit) {
-            const int who = __ffs(hit) - 1;
-            row = r0 + who;
-            t0 = __shfl_sync(0xffffffffu, start, who);
-            n_new = __shfl_sync(0xffffffffu, count, who);
-            c0 = (s - (t0 / TC + row)) * TC;
-            return true;
-        }
-    }
-    return false;
-}
-
 // Inclusive sums of log_a over the chunk's tokens into Ls[TC], b into bs[TC] (zero beyond the
 // chunk's tokens), by the CTA's first warp.
 __device__ __forceinline__ void chunk_gates(const ScanArgs& a, int64_t n0, int nt, int head,
                                             float* Ls, float* bs) {
     if (threadIdx.x >= 32) return;
     const int lane = threadIdx.x;
-    const int64_t at = (n0 + 2 * lane) * a.H + head;
+    const int64_t at = (n0 + 2 * lane) * a.ld_gates + head;
     const float x0 = 2 * lane < nt ? a.log_a[at] : 0.f;
-    const float x1 = 2 * lane + 1 < nt ? a.log_a[at + a.H] : 0.f;
-    bs[2 * lane] = 2 * lane < nt ? a.b[at] : 0.f;
-    bs[2 * lane + 1] = 2 * lane + 1 < nt ? a.b[at + a.H] : 0.f;
+    const float x1 = 2 * lane + 1 < nt ? a.log_a[at + a.ld_gates] : 0.f;
+    const float* b = a.b ? a.b + (n0 + 2 * lane) * a.H + head : nullptr;
+    bs[2 * lane] = 2 * lane < nt ? (b ? b[0] : 1.f) : 0.f;
+    bs[2 * lane + 1] = 2 * lane + 1 < nt ? (b ? b[a.H] : 1.f) : 0.f;
     float sum = x0 + x1;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
@@ -330,7 +306,7 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(const ScanArgs a) {
     pdl_wait();
     pdl_trigger();
     int row, t0, c0, n_new;
-    if (!find_chunk(a, blockIdx.x, row, t0, c0, n_new)) return;
+    if (!find_chunk(a.row_start, a.n_rows, a.min_chunked, blockIdx.x, row, t0, c0, n_new)) return;
     const int head = blockIdx.y, v0 = blockIdx.z * VB;
     const int N = a.N, V = a.V, H = a.H;
     const int nt = min(TC, n_new - c0);
@@ -475,7 +451,7 @@ __global__ void __launch_bounds__(256, 3) chunk_out_kernel(const ScanArgs a) {
     pdl_wait();
     pdl_trigger();
     int row, t0, c0, n_new;
-    if (!find_chunk(a, blockIdx.x, row, t0, c0, n_new)) return;
+    if (!find_chunk(a.row_start, a.n_rows, a.min_chunked, blockIdx.x, row, t0, c0, n_new)) return;
     const int head = blockIdx.y, v0 = blockIdx.z * VB;
     const int N = a.N, V = a.V, H = a.H;
     const int nt = min(TC, n_new - c0);
@@ -658,7 +634,9 @@ SLLM_EXPORT int sllm_gated_scan_chunks_fit(int N, int V) {
     return N % 16 == 0 && N <= CHUNK_MAX_N && V % 8 == 0;
 }
 
-// q, k: [n_tokens, >= G N], v: [n_tokens, >= H V] (dtype), log_a, b: float [n_tokens, H]; state:
+// q, k: [n_tokens, >= G N], v: [n_tokens, >= H V] (dtype), log_a, b: float [n_tokens, H] (ld_gates H;
+// ld_gates 0: log_a [H]; b may be null: 1); silu: q, k and v are taken through a silu (not with
+// chunked); state:
 // float [slots, H, V + ones, N]; out: float [n_tokens, H V]; ones_out: float [n_tokens, H] (ones
 // only); skip: float [H] or null.  chunked: rows of at least min_chunked tokens take the chunk
 // kernels, with the scratch dS float [n_tokens / 64 + n_rows + 1, H, V + ones, N] and decay float
@@ -666,6 +644,7 @@ SLLM_EXPORT int sllm_gated_scan_chunks_fit(int N, int V) {
 // a row brings.
 SLLM_EXPORT int sllm_gated_scan(const void* q, int64_t ldq, const void* k, int64_t ldk,
                                 const void* v, int64_t ldv, const float* log_a, const float* b,
+                                int64_t ld_gates, int silu,
                                 float* state, const int* row_start, const int* row_slot,
                                 float* out, float* ones_out, const float* skip, float scale,
                                 int n_tokens, int n_rows, int H, int G, int N, int V, int ones,
@@ -674,11 +653,12 @@ SLLM_EXPORT int sllm_gated_scan(const void* q, int64_t ldq, const void* k, int64
     if (n_tokens <= 0 || n_rows <= 0) return 0;
     if (H < 1 || G < 1 || H % G || N < 1 || N > 1024 || V < 1 || ones < 0 || ones > 1 ||
         (ones && !ones_out) || ldq < (int64_t)G * N || ldk < (int64_t)G * N ||
-        ldv < (int64_t)H * V || H > 65535 || n_rows > 65535 || dtype < 0 || dtype > 1)
+        ldv < (int64_t)H * V || H > 65535 || n_rows > 65535 || dtype < 0 || dtype > 1 ||
+        (ld_gates != 0 && ld_gates != H) || (silu && chunked))
         return (int)cudaErrorInvalidValue;
     const int vec4 = !((ldq | ldk | N) & 3) && !(((uintptr_t)q | (uintptr_t)k) & 15);
-    ScanArgs a = {q, ldq, k, ldk, v, ldv, log_a, b, state, row_start, row_slot, out, ones_out, skip,
-                  scale, H, G, N, V, V + ones, vec4, 0x7fffffff, dS, decay, n_rows};
+    ScanArgs a = {q, ldq, k, ldk, v, ldv, log_a, b, ld_gates, state, row_start, row_slot, out, ones_out,
+                  skip, scale, H, G, N, V, V + ones, vec4, silu, 0x7fffffff, dS, decay, n_rows};
     if ((N & 3) == 0 && ((uintptr_t)state & 15)) return (int)cudaErrorInvalidValue;
     if (chunked) {
         if (dtype != 1 || !dS || !decay || min_chunked < 1 || !sllm_gated_scan_chunks_fit(N, V) ||

@@ -13,6 +13,9 @@
 // k0 + 8t + 7] and W[row g + 8][same k], which feeds two m16n8k16 products if the B fragments
 // (the tokens' activations) are read with the same permutation of k.  The eight partial sums of
 // a CTA are added in warp order, so a token's result does not depend on the batch.
+//
+// Several products of equal sizes may share a launch (groups along y): group g multiplies its own
+// activations by its own matrix, each a fixed number of elements behind the group before.
 #include "common.cuh"
 
 namespace sllm {
@@ -46,7 +49,10 @@ template <int MT, bool SWIGLU, typename TOut>
 __global__ void __launch_bounds__(GV_THREADS)
 gemv_mma_kernel(const bf16* __restrict__ X, const bf16* __restrict__ W, TOut* __restrict__ Y,
                 int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldy, int act, float act_p0,
-                float act_p1) {
+                float act_p1, int64_t group_x, int64_t group_w, int64_t group_y) {
+    X += blockIdx.y * group_x;
+    W += blockIdx.y * group_w;
+    Y += blockIdx.y * group_y;
     constexpr int NW = SWIGLU ? 2 : 1;
     __shared__ float red[GV_WARPS][GV_ROWS][8 * MT + 1];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -183,13 +189,15 @@ static int g_gemv_pdl = 1;
 
 template <int MT, bool SWIGLU, typename TOut>
 static int launch_gemv(const void* X, const void* W, void* Y, int M, int N, int K, int64_t ldx,
-                       int64_t ldw, int64_t ldy, int act, float p0, float p1, cudaStream_t stream) {
+                       int64_t ldw, int64_t ldy, int act, float p0, float p1, cudaStream_t stream,
+                       int groups = 1, int64_t group_x = 0, int64_t group_w = 0,
+                       int64_t group_y = 0) {
     const int n_out = SWIGLU ? N / 2 : N;
     const int grid = (n_out + GV_ROWS - 1) / GV_ROWS;
     // launched so that it may start while the previous kernel of the stream drains: the kernel
     // requests its first weights, then waits for that kernel (pdl_wait) before it reads X
     cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(grid);
+    cfg.gridDim = dim3(grid, groups);
     cfg.blockDim = dim3(GV_THREADS);
     cfg.dynamicSmemBytes = 0;
     cfg.stream = stream;
@@ -199,7 +207,8 @@ static int launch_gemv(const void* X, const void* W, void* Y, int M, int N, int 
     cfg.attrs = attr;
     cfg.numAttrs = 1;
     cudaError_t e = cudaLaunchKernelEx(&cfg, gemv_mma_kernel<MT, SWIGLU, TOut>, (const bf16*)X,
-                                       (const bf16*)W, (TOut*)Y, M, N, K, ldx, ldw, ldy, act, p0, p1);
+                                       (const bf16*)W, (TOut*)Y, M, N, K, ldx, ldw, ldy, act, p0, p1,
+                                       group_x, group_w, group_y);
     if (e != cudaSuccess) return (int)e;
     return 0;
 }
@@ -242,5 +251,24 @@ SLLM_EXPORT int sllm_gemv_mma(const void* X, const void* W, void* Y, int M, int 
         if (out_dtype == 1) return pick_mt<false, bf16>(X, W, Y, M, N, K, ldx, ldw, ldy, 0, 0.f, 0.f, stream);
         if (out_dtype == 0) return pick_mt<false, float>(X, W, Y, M, N, K, ldx, ldw, ldy, 0, 0.f, 0.f, stream);
     }
+    return (int)cudaErrorInvalidValue;
+}
+
+// `groups` plain products of up to 8 tokens: Y_g [M, N] = X_g [M, K] W_g [N, K]^T, where group g's
+// activations, matrix and output start g * group_x / group_w / group_y elements behind X / W / Y.
+SLLM_EXPORT int sllm_gemv_mma_groups(const void* X, const void* W, void* Y, int groups, int M, int N,
+                                     int K, int64_t ldx, int64_t ldw, int64_t ldy, int64_t group_x,
+                                     int64_t group_w, int64_t group_y, int out_dtype,
+                                     cudaStream_t stream) {
+    if (M <= 0 || N <= 0 || groups <= 0) return 0;
+    if (M > 8 || groups > 65535 || K <= 0 ||
+        ((K | ldx | ldw | group_x | group_w) & 7) || (((uintptr_t)X | (uintptr_t)W) & 15))
+        return (int)cudaErrorInvalidValue;
+    if (out_dtype == 1)
+        return launch_gemv<1, false, bf16>(X, W, Y, M, N, K, ldx, ldw, ldy, 0, 0.f, 0.f, stream, groups,
+                                           group_x, group_w, group_y);
+    if (out_dtype == 0)
+        return launch_gemv<1, false, float>(X, W, Y, M, N, K, ldx, ldw, ldy, 0, 0.f, 0.f, stream,
+                                            groups, group_x, group_w, group_y);
     return (int)cudaErrorInvalidValue;
 }

@@ -3,6 +3,7 @@
 //
 //   x[n]   = resid[n] + sum_i coef_i * term_i[n]          (up to LN_MAX_TERMS terms, in order)
 //   out[n] = (x[n] - mean) / sqrt(var + eps) * w + b,     var = mean((x - mean)^2)
+//   (b may be null: no offset)
 //
 // The stream is 32-bit and all of the arithmetic is; the terms are branch outputs in the
 // compute dtype.  Without out_rows every token is normed and the stream is updated in place;
@@ -55,7 +56,7 @@ add_layernorm_kernel(float* resid, const LnTerms terms, const float* __restrict_
     const float inv = 1.0f / sqrtf(block_sum(dev, scratch) / (float)d + eps);
     TO* o = out + (int64_t)blockIdx.x * d;
     for (int c = threadIdx.x; c < d; c += LN_THREADS)
-        o[c] = from_float<TO>((row[c] - mean) * inv * w[c] + b[c]);
+        o[c] = from_float<TO>((row[c] - mean) * inv * w[c] + (b ? b[c] : 0.f));
 }
 
 // Four elements at a time (d a multiple of 4, every base 16-byte aligned): the same sums in
@@ -110,7 +111,8 @@ add_layernorm_vec_kernel(float* resid, const LnTerms terms, const float* __restr
     const float inv = 1.0f / sqrtf(block_sum(dev, scratch) / (float)d + eps);
     TO* o = out + (int64_t)blockIdx.x * d;
     for (int c = threadIdx.x * 4; c < d; c += LN_THREADS * 4) {
-        const float4 x = load4(row + c), g = load4(w + c), h = load4(b + c);
+        const float4 x = load4(row + c), g = load4(w + c);
+        const float4 h = b ? load4(b + c) : make_float4(0.f, 0.f, 0.f, 0.f);
         store4(o + c, make_float4((x.x - mean) * inv * g.x + h.x, (x.y - mean) * inv * g.y + h.y,
                                   (x.z - mean) * inv * g.z + h.z, (x.w - mean) * inv * g.w + h.w));
     }

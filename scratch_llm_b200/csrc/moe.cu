@@ -5,7 +5,7 @@
 //            (score + correction), groups of neighbouring outputs of which only the best
 //            `keep` (by their largest choice score) stay eligible, the `top` largest choice
 //            scores (ties: the lower index), weights = the chosen outputs' scores over their
-//            sum (+ 1e-20).  Outputs from n_real on are identity experts: they need no
+//            sum (+ 1e-20), times a constant.  Outputs from n_real on are identity experts: they need no
 //            product.  Counts the tokens of every real expert.
 //   plan     offsets of the experts' token lists and the list of row tiles (expert, first
 //            row, rows) that the grouped products walk.
@@ -37,7 +37,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z,
                                             int n_total, int n_real, int n_groups, int keep,
                                             int top, int lane, int* __restrict__ ids_row,
                                             float* __restrict__ weights_row, int* counts,
-                                            int flags) {
+                                            int flags, float weight_scale) {
     float* choice = score + n_total;   // score + correction, -inf once taken or barred
     if (flags & MOE_SIGMOID) {
         for (int e = lane; e < n_total; e += 32) {
@@ -147,7 +147,8 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z,
     }
     if (lane < top) {
         ids_row[lane] = my_id;
-        weights_row[lane] = (flags & MOE_RAW_WEIGHTS) ? my_w : my_w / (wsum + 1e-20f);
+        weights_row[lane] =
+            weight_scale * ((flags & MOE_RAW_WEIGHTS) ? my_w : my_w / (wsum + 1e-20f));
         if (my_id >= 0 && my_id < n_real) atomicAdd(&counts[my_id], 1);
     }
 }
@@ -159,7 +160,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ldl,
                                  const int* __restrict__ token_row, int N, int n_total,
                                  int n_real, int n_groups, int keep, int top,
                                  int* __restrict__ ids, float* __restrict__ weights,
-                                 int* __restrict__ counts, int flags) {
+                                 int* __restrict__ counts, int flags, float weight_scale) {
     pdl_wait();
     pdl_trigger();
     extern __shared__ float smem[];
@@ -175,7 +176,8 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ldl,
     }
     route_token(logits + (int64_t)n * ldl, corr,
                 smem + (size_t)warp * (2 * n_total + 2 * n_groups), n_total, n_real, n_groups, keep,
-                top, lane, ids + (int64_t)n * top, weights + (int64_t)n * top, counts, flags);
+                top, lane, ids + (int64_t)n * top, weights + (int64_t)n * top, counts, flags,
+                weight_scale);
 }
 
 // Steps of few tokens (decode): ONE CTA routes every token, counts, plans the tiles, gives every
@@ -192,7 +194,7 @@ moe_route_small_kernel(const float* __restrict__ logits, int64_t ldl,
                        float* __restrict__ weights, int* __restrict__ meta, int max_tiles,
                        int tile_rows, int* __restrict__ pair_token, int* __restrict__ pair_place,
                        const __nv_bfloat16* __restrict__ x, int64_t ldx, int K,
-                       __nv_bfloat16* __restrict__ rows_out, int flags) {
+                       __nv_bfloat16* __restrict__ rows_out, int flags, float weight_scale) {
     pdl_wait();
     pdl_trigger();
     extern __shared__ float smem[];
@@ -215,7 +217,8 @@ moe_route_small_kernel(const float* __restrict__ logits, int64_t ldl,
         }
         route_token(logits + (int64_t)n * ldl, corr, smem + (size_t)warp * per_warp, n_total,
                     n_real, n_groups, keep, top, lane, ids + (int64_t)n * top,
-                    weights + (int64_t)n * top, counts, flags);
+                    weights + (int64_t)n * top, counts, flags,
+                weight_scale);
     }
     __syncthreads();
     for (int e = tid; e <= n_real; e += blockDim.x) {
@@ -488,7 +491,7 @@ SLLM_EXPORT int sllm_moe_route(const float* logits, int64_t ldl, const float* co
                                int n_tokens, int n_total, int n_real, int n_groups, int keep,
                                int top, int* ids, float* weights, int* work, int max_tiles,
                                int tile_rows, int* pair_token, int* pair_place, int flags,
-                               cudaStream_t stream) {
+                               float weight_scale, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (n_total <= 0 || ldl < n_total || n_real < 0 || n_real > n_total || top < 1 ||
         top > MOE_MAX_TOP || top > n_total || n_groups < 1 || n_total % n_groups || keep < 1 || keep > n_groups ||
@@ -503,7 +506,7 @@ SLLM_EXPORT int sllm_moe_route(const float* logits, int64_t ldl, const float* co
                                       dim3(32 * warps),
                                       (size_t)warps * (2 * n_total + 2 * n_groups) * sizeof(float),
                                       stream, logits, ldl, corr, token_row, n_tokens, n_total, n_real,
-                                      n_groups, keep, top, ids, weights, counts, flags);
+                                      n_groups, keep, top, ids, weights, counts, flags, weight_scale);
     if (err != cudaSuccess) return (int)err;
     if (n_real == 0) return 0;
     err = sllm_launch_pdl(moe_plan_kernel, dim3(1), dim3(256), 0, stream, (const int*)counts,
@@ -528,7 +531,7 @@ SLLM_EXPORT int sllm_moe_route_small(const float* logits, int64_t ldl, const flo
                                      int top, int* ids, float* weights, int* meta, int max_tiles,
                                      int tile_rows, int* pair_token, int* pair_place,
                                      const void* x, int64_t ldx, int K, void* rows_out, int flags,
-                                     cudaStream_t stream) {
+                                     float weight_scale, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (n_total <= 0 || ldl < n_total || n_real < 0 || n_real > n_total || top < 1 ||
         top > MOE_MAX_TOP || top > n_total || n_groups < 1 || n_total % n_groups || keep < 1 || keep > n_groups ||
@@ -543,7 +546,7 @@ SLLM_EXPORT int sllm_moe_route_small(const float* logits, int64_t ldl, const flo
                                 (size_t)smem, stream, logits, ldl, corr, token_row, n_tokens, n_total,
                                 n_real, n_groups, keep, top, ids, weights, meta, max_tiles,
                                 tile_rows, pair_token, pair_place, (const __nv_bfloat16*)x, ldx, K,
-                                (__nv_bfloat16*)rows_out, flags);
+                                (__nv_bfloat16*)rows_out, flags, weight_scale);
 }
 
 // dtype: 0 = float32 operands, 1 = bfloat16 operands.  gated 1 (silu(gate) * up) and 2 (squared

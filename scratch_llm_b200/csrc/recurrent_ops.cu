@@ -348,12 +348,18 @@ lowrank_decay_kernel(const float* __restrict__ pre, int64_t ldp, const float* __
 //     mode 0:  out = z
 //     mode 1:  out = -exp(rate_log[c / per_rate]) * softplus(z)    (the logarithm of a decay
 //              exp(-exp(A) softplus(z)) with one A per `per_rate` channels)
+//     mode 2:  out = rate * log sigmoid(z)                         (of a decay sigmoid(z)^rate)
+//     mode 3:  out = -exp(z)                                       (of a decay exp(-exp(z)))
+// In modes 2 and 3 out is at least LOG_DECAY_FLOOR: beyond it a state is zero in 32-bit within a
+// token, and sums of such logarithms keep their precision.  tanh_in: the hidden values pass a tanh.
 // The sum runs over r in ascending order for every token, whatever the batch.  out: [N, C],
 // float32 or bfloat16.  One launch serves up to two such products of the same `pre` (a mixer's
 // decays and its gate): the first `blocks0` CTAs along x take the first job, the rest the second.
 // grid (blocks of both jobs, ceil(N / LOWRANK_TOKENS)); shared: LOWRANK_TOKENS * max R floats.
+constexpr float LOG_DECAY_FLOOR = -88.f;
 struct ExpandJob {
     int col0; const float* w2t; const float* bias; const float* rate_log; int per_rate; int mode;
+    float rate; int tanh_in;
     void* out; int out_bf16; int C; int R;
 };
 
@@ -370,7 +376,8 @@ lowrank_expand_kernel(const float* __restrict__ pre, int64_t ldp, const ExpandJo
     const int nt = min(LOWRANK_TOKENS, N - n0);
     for (int i = threadIdx.x; i < LOWRANK_TOKENS * R; i += blockDim.x) {
         const int t = i / R, r = i - t * R;
-        th[t * R + r] = t < nt ? pre[(int64_t)(n0 + t) * ldp + j.col0 + r] : 0.f;
+        const float h = t < nt ? pre[(int64_t)(n0 + t) * ldp + j.col0 + r] : 0.f;
+        th[t * R + r] = j.tanh_in ? tanhf(h) : h;
     }
     __syncthreads();
     const int c = ((int)blockIdx.x - (second ? blocks0 : 0)) * blockDim.x + threadIdx.x;
@@ -400,6 +407,9 @@ lowrank_expand_kernel(const float* __restrict__ pre, int64_t ldp, const ExpandJo
         if (t < nt) {
             float z = acc[t] + b0;
             if (j.mode == 1) z = -rate * (z > 20.f ? z : log1pf(expf(z)));
+            else if (j.mode == 2)
+                z = fmaxf(j.rate * (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))), LOG_DECAY_FLOOR);
+            else if (j.mode == 3) z = fmaxf(-expf(z), LOG_DECAY_FLOOR);
             const int64_t at = (int64_t)(n0 + t) * C + c;
             if (j.out_bf16) reinterpret_cast<__nv_bfloat16*>(j.out)[at] = __float2bfloat16_rn(z);
             else reinterpret_cast<float*>(j.out)[at] = z;
@@ -407,15 +417,16 @@ lowrank_expand_kernel(const float* __restrict__ pre, int64_t ldp, const ExpandJo
     }
 }
 
-// The gate ahead of the norm: y = o * silu(gate), then each of `parts` equal parts of y over its
-// own root mean square, times gain [W].  o: float [n_tokens, W]; one CTA per (token, part), a
+// The gate ahead of the norm: y = o * act(gate), then each of `parts` equal parts of y over its
+// own root mean square, times gain [W]; or (after) the norm of o first, then the gate: out = o over
+// its part's root mean square, times gain, times act(gate).  gate_act: 0 = silu, 1 = sigmoid.  o: float [n_tokens, W]; one CTA per (token, part), a
 // part of P = W / parts elements waits in shared memory between the two passes.  V: elements per
 // access (4 where P and the rows allow 16-byte reads of o, else 1).
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
 gate_part_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, int64_t ldg,
                       const float* __restrict__ gain, float eps, T* __restrict__ out, int64_t ldo,
-                      int W, int P) {
+                      int W, int P, int gate_act, int after) {
     pdl_wait();
     pdl_trigger();
     extern __shared__ __align__(16) float gp_row[];     // [P]
@@ -426,10 +437,13 @@ gate_part_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, i
     for (int i = threadIdx.x * V; i < P; i += blockDim.x * V) {
         float v[V], z[V];
         load_few<V>(o + n * W + at + i, v);
-        load_few<V>(gate + n * ldg + at + i, z);
+        if (!after) {
+            load_few<V>(gate + n * ldg + at + i, z);
+#pragma unroll
+            for (int k = 0; k < V; ++k) v[k] *= (gate_act ? 1.f : z[k]) * sigmoid_of<T>(z[k]);
+        }
 #pragma unroll
         for (int k = 0; k < V; ++k) {
-            v[k] *= z[k] * sigmoid_of<T>(z[k]);
             ss = fmaf(v[k], v[k], ss);
             gp_row[i + k] = v[k];
         }
@@ -440,6 +454,12 @@ gate_part_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, i
         float v[V];
 #pragma unroll
         for (int k = 0; k < V; ++k) v[k] = gp_row[i + k] * inv * gain[at + i + k];
+        if (after) {
+            float z[V];
+            load_few<V>(gate + n * ldg + at + i, z);
+#pragma unroll
+            for (int k = 0; k < V; ++k) v[k] *= (gate_act ? 1.f : z[k]) * sigmoid_of<T>(z[k]);
+        }
         store_few<V>(out + n * ldo + at + i, v);
     }
 }
@@ -541,6 +561,83 @@ __global__ void __launch_bounds__(256) memory_gates_kernel(const MemoryGates a) 
         for (int w = 0; w < 8; ++w) carried = fmaxf(wF[w] + carried, wM[w]);
     }
     if (tid == 0) *m = carried;
+}
+
+// A token shift in front of several projections: with h' the previous token's h (a row's first
+// token: what the slot carries, zeros at a sequence's start), out[m, n, :] = h + (h' - h) * mu[m] for
+// m = 0 .. M - 1.  The row's last h is left in the slot by whoever takes the row's first token, after
+// the old one has been read.  h [n_tokens, d], mu [M, d], state [slots, d] (32-bit), out [M, n_tokens,
+// d].  A thread takes V channels of SHIFT_RUN consecutive tokens.  Padding tokens (row -1) get zeros.
+constexpr int SHIFT_RUN = 4;
+template <typename T, int V>
+__global__ void __launch_bounds__(128)
+shift_mix_kernel(const T* __restrict__ h, int64_t ldh, const float* __restrict__ mu, int M,
+                 float* __restrict__ state, const int* __restrict__ token_row,
+                 const int* __restrict__ row_start, const int* __restrict__ row_slot,
+                 T* __restrict__ out, int d, int n_tokens) {
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+    pdl_wait();
+    pdl_trigger();
+    if (c >= d) return;
+    const int n0 = blockIdx.y * SHIFT_RUN;
+    float now[SHIFT_RUN][V], before[SHIFT_RUN][V];
+    int rows[SHIFT_RUN];
+#pragma unroll
+    for (int i = 0; i < SHIFT_RUN; ++i) {
+        rows[i] = n0 + i < n_tokens ? token_row[n0 + i] : -1;
+#pragma unroll
+        for (int k = 0; k < V; ++k) now[i][k] = before[i][k] = 0.f;
+        if (rows[i] >= 0) load_few<V>(h + (int64_t)(n0 + i) * ldh + c, now[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < SHIFT_RUN; ++i) {
+        const int r = rows[i], n = n0 + i;
+        if (r < 0) continue;
+        if (n > row_start[r]) {
+            if (i) {
+#pragma unroll
+                for (int k = 0; k < V; ++k) before[i][k] = now[i ? i - 1 : 0][k];
+            } else {
+                load_few<V>(h + (int64_t)(n - 1) * ldh + c, before[i]);
+            }
+        } else {
+            float* mine = state + (int64_t)row_slot[r] * d + c;
+            float last[V];
+            load_few<V>(mine, before[i]);
+            load_few<V>(h + (int64_t)(row_start[r + 1] - 1) * ldh + c, last);
+            store_few<V>(mine, last);
+        }
+    }
+    for (int m = 0; m < M; ++m) {
+        float w[V];
+        load_few<V>(mu + (int64_t)m * d + c, w);
+#pragma unroll
+        for (int i = 0; i < SHIFT_RUN; ++i) {
+            if (n0 + i >= n_tokens) break;
+            float x[V];
+#pragma unroll
+            for (int k = 0; k < V; ++k) x[k] = fmaf(before[i][k] - now[i][k], w[k], now[i][k]);
+            store_few<V>(out + ((int64_t)m * n_tokens + n0 + i) * d + c, x);
+        }
+    }
+}
+
+// silu in place on the first C columns of x's rows.
+template <typename T, int V>
+__global__ void silu_columns_kernel(T* __restrict__ x, int64_t ldx, int C, int64_t n_items) {
+    pdl_wait();
+    pdl_trigger();
+    const int per_row = C / V;
+    for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < n_items;
+         i += (int64_t)gridDim.x * blockDim.x) {
+        const int64_t n = i / per_row;
+        T* p = x + n * ldx + (i - n * per_row) * V;
+        float z[V];
+        load_few<V>(p, z);
+#pragma unroll
+        for (int k = 0; k < V; ++k) z[k] *= sigmoid_of<T>(z[k]);
+        store_few<V>(p, z);
+    }
 }
 
 }  // namespace sllm
@@ -649,12 +746,13 @@ SLLM_EXPORT int sllm_lowrank_decay(const float* pre, int64_t ldp, const float* w
 }
 
 // Up to two products of one `pre` in a launch (n_jobs 1 or 2); per job: col0, w2t [R, C], bias
-// (may be null), rate_log with per_rate (mode 1), mode, out [N, C], out_dtype (0 = float32,
+// (may be null), rate_log with per_rate (mode 1), rate (mode 2), tanh_in, mode, out [N, C], out_dtype (0 = float32,
 // 1 = bfloat16), C, R.
 SLLM_EXPORT int sllm_lowrank_expand(const float* pre, int64_t ldp, int n_jobs, const int* col0,
                                     const float* const* w2t, const float* const* bias,
                                     const float* const* rate_log, const int* per_rate,
-                                    const int* mode, void* const* out, const int* out_dtype,
+                                    const float* rates, const int* tanh_in, const int* mode,
+                                   void* const* out, const int* out_dtype,
                                     const int* C, const int* R, int n_tokens,
                                     cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
@@ -663,11 +761,12 @@ SLLM_EXPORT int sllm_lowrank_expand(const float* pre, int64_t ldp, int n_jobs, c
     int max_r = 0, max_c = 0;
     for (int i = 0; i < n_jobs; ++i) {
         if (C[i] <= 0 || R[i] <= 0 || R[i] > 1024 || col0[i] < 0 || ldp < col0[i] + R[i] ||
-            mode[i] < 0 || mode[i] > 1 || out_dtype[i] < 0 || out_dtype[i] > 1 ||
+            mode[i] < 0 || mode[i] > 3 || out_dtype[i] < 0 || out_dtype[i] > 1 ||
             (mode[i] == 1 && (!rate_log[i] || per_rate[i] <= 0 || C[i] % per_rate[i])))
             return (int)cudaErrorInvalidValue;
         j[i].col0 = col0[i]; j[i].w2t = w2t[i]; j[i].bias = bias[i]; j[i].rate_log = rate_log[i];
         j[i].per_rate = per_rate[i]; j[i].mode = mode[i]; j[i].out = out[i];
+        j[i].rate = rates[i]; j[i].tanh_in = tanh_in[i];
         j[i].out_bf16 = out_dtype[i]; j[i].C = C[i]; j[i].R = R[i];
         max_r = R[i] > max_r ? R[i] : max_r;
         max_c = C[i] > max_c ? C[i] : max_c;
@@ -684,14 +783,16 @@ SLLM_EXPORT int sllm_lowrank_expand(const float* pre, int64_t ldp, int n_jobs, c
     return 0;
 }
 
-// out = parts of o * silu(gate) over their root mean squares, times gain.  o: float [n_tokens, W];
-// gate / out: rows ldg / ldo apart.
+// out = parts of o * act(gate) over their root mean squares, times gain; after: parts of o over
+// their root mean squares, times gain, times act(gate).  gate_act 0 = silu, 1 = sigmoid.  o: float
+// [n_tokens, W]; gate / out: rows ldg / ldo apart.
 SLLM_EXPORT int sllm_gate_part_norm(const float* o, const void* gate, int64_t ldg,
                                     const float* gain, float eps, void* out, int64_t ldo,
-                                    int n_tokens, int W, int parts, int dtype,
-                                    cudaStream_t stream) {
+                                    int n_tokens, int W, int parts, int gate_act, int after,
+                                    int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (W <= 0 || parts < 1 || parts > 65535 || W % parts || ldg < W || ldo < W)
+    if (W <= 0 || parts < 1 || parts > 65535 || W % parts || ldg < W || ldo < W ||
+        gate_act < 0 || gate_act > 1)
         return (int)cudaErrorInvalidValue;
     const int P = W / parts;
     const size_t smem = (size_t)P * sizeof(float);
@@ -709,7 +810,7 @@ SLLM_EXPORT int sllm_gate_part_norm(const float* o, const void* gate, int64_t ld
         }                                                                                        \
         return (int)sllm_launch_pdl(gate_part_norm_kernel<T, V>, dim3(n_tokens, parts),          \
                                     dim3(256), smem, stream, o, (const T*)gate, ldg, gain, eps,  \
-                                    (T*)out, ldo, W, P);                                         \
+                                    (T*)out, ldo, W, P, gate_act, after);                                         \
     } while (0)
     if (dtype == 0 && vec) SLLM_GPN(float, 4);
     if (dtype == 0) SLLM_GPN(float, 1);
@@ -744,4 +845,48 @@ SLLM_EXPORT int sllm_memory_gates(const float* pre, int64_t ldp, const float* bi
         return (int)sllm_launch_pdl(memory_gates_step_kernel, dim3((n_rows * H + 127) / 128),
                                     dim3(128), 0, stream, a, n_rows);
     return (int)sllm_launch_pdl(memory_gates_kernel, dim3(H, n_rows), dim3(256), 0, stream, a);
+}
+
+// h: [n_tokens, >= d] (dtype), mu: float [M, d], state: float [slots, d], out: [M, n_tokens, d] (dtype).
+SLLM_EXPORT int sllm_shift_mix(const void* h, int64_t ldh, const float* mu, int M, float* state,
+                               const int* token_row, const int* row_start, const int* row_slot,
+                               void* out, int n_tokens, int d, int dtype, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    const int runs = (n_tokens + SHIFT_RUN - 1) / SHIFT_RUN;
+    if (d <= 0 || M < 1 || ldh < d || runs > 65535) return (int)cudaErrorInvalidValue;
+    const bool vec = ((d | ldh) & 3) == 0 &&
+                     !(((uintptr_t)h | (uintptr_t)mu | (uintptr_t)state | (uintptr_t)out) & 15);
+    const int per = vec ? 4 : 1;
+    const dim3 grid((d / per + 127) / 128, runs);
+    typedef __nv_bfloat16 bf16;
+#define SLLM_SM(T, V)                                                                              \
+    return (int)sllm_launch_pdl(shift_mix_kernel<T, V>, grid, dim3(128), 0, stream, (const T*)h,   \
+                                ldh, mu, M, state, token_row, row_start, row_slot, (T*)out, d,     \
+                                n_tokens)
+    if (dtype == 0 && vec) SLLM_SM(float, 4);
+    if (dtype == 0) SLLM_SM(float, 1);
+    if (dtype == 1 && vec) SLLM_SM(bf16, 4);
+    if (dtype == 1) SLLM_SM(bf16, 1);
+#undef SLLM_SM
+    return (int)cudaErrorInvalidValue;
+}
+
+SLLM_EXPORT int sllm_silu_columns(void* x, int64_t ldx, int n_tokens, int C, int dtype,
+                                  cudaStream_t stream) {
+    if (n_tokens <= 0 || C == 0) return 0;
+    if (C < 0 || ldx < C) return (int)cudaErrorInvalidValue;
+    const bool vec = ((C | ldx) & 3) == 0 && !((uintptr_t)x & 15);
+    const int64_t items = (int64_t)n_tokens * (vec ? C / 4 : C);
+    int64_t blocks = (items + 255) / 256;
+    if (blocks > 148 * 32) blocks = 148 * 32;
+    typedef __nv_bfloat16 bf16;
+#define SLLM_SC(T, V)                                                                              \
+    return (int)sllm_launch_pdl(silu_columns_kernel<T, V>, dim3((int)blocks), dim3(256), 0, stream, \
+                                (T*)x, ldx, C, items)
+    if (dtype == 0 && vec) SLLM_SC(float, 4);
+    if (dtype == 0) SLLM_SC(float, 1);
+    if (dtype == 1 && vec) SLLM_SC(bf16, 4);
+    if (dtype == 1) SLLM_SC(bf16, 1);
+#undef SLLM_SC
+    return (int)cudaErrorInvalidValue;
 }

@@ -11,7 +11,7 @@
 // the listed tokens are normed (outA is then [rows, d]) and the stream is not written.
 // One CTA per token; the row waits in shared memory between the two passes, so a token's result
 // does not depend on its neighbours.
-#include "common.cuh"
+#include "few.cuh"
 
 namespace sllm {
 
@@ -20,52 +20,11 @@ constexpr int SN_MAX_TERMS = 4;
 struct SumNorm {
     float* resid;
     const void* term[SN_MAX_TERMS]; float coef[SN_MAX_TERMS]; int n_terms;
-    // the routed sum (y null: none): y [places, d], ids / weights / place [tokens, top]
-    const float* y; const int* ids; const float* weights; const int* place; int top;
-    const void* shared; const float* sg; int64_t ldsg;     // shared, sg may be null
+    RoutedRows routed;
     const float* gA; const float* gB; float eps;
     void* outA; void* outB;
     const int* out_rows; int d;
 };
-
-template <int V> struct Few { float v[V]; };
-template <int V> __device__ __forceinline__ Few<V> few(const float* p) {
-    Few<V> r;
-    if (V == 4) {
-        const float4 x = *reinterpret_cast<const float4*>(p);
-        r.v[0] = x.x; r.v[V - 3] = x.y; r.v[V - 2] = x.z; r.v[V - 1] = x.w;
-    } else {
-        r.v[0] = *p;
-    }
-    return r;
-}
-template <int V> __device__ __forceinline__ Few<V> few(const __nv_bfloat16* p) {
-    Few<V> r;
-    if (V == 4) {
-        const uint2 x = *reinterpret_cast<const uint2*>(p);
-        const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&x);
-        r.v[0] = __low2float(h[0]); r.v[V - 3] = __high2float(h[0]);
-        r.v[V - 2] = __low2float(h[1]); r.v[V - 1] = __high2float(h[1]);
-    } else {
-        r.v[0] = __bfloat162float(*p);
-    }
-    return r;
-}
-template <int V> __device__ __forceinline__ void put(float* p, const Few<V>& r) {
-    if (V == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[V - 3], r.v[V - 2], r.v[V - 1]);
-    else *p = r.v[0];
-}
-template <int V> __device__ __forceinline__ void put(__nv_bfloat16* p, const Few<V>& r) {
-    if (V == 4) {
-        uint2 x;
-        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&x);
-        h[0] = __floats2bfloat162_rn(r.v[0], r.v[V - 3]);
-        h[1] = __floats2bfloat162_rn(r.v[V - 2], r.v[V - 1]);
-        *reinterpret_cast<uint2*>(p) = x;
-    } else {
-        *p = __float2bfloat16_rn(r.v[0]);
-    }
-}
 
 template <typename T, int V>
 __global__ void __launch_bounds__(512) sum_norm_kernel(const SumNorm a) {
@@ -76,9 +35,8 @@ __global__ void __launch_bounds__(512) sum_norm_kernel(const SumNorm a) {
     const int d = a.d;
     const int64_t n = a.out_rows ? a.out_rows[blockIdx.x] : blockIdx.x;
     float* r = a.resid + n * d;
-    const bool keep = a.out_rows == nullptr && (a.n_terms > 0 || a.y != nullptr);
-    float fs = 1.f;
-    if (a.y && a.shared && a.sg) fs = 1.0f / (1.0f + expf(-a.sg[n * a.ldsg]));
+    const bool keep = a.out_rows == nullptr && (a.n_terms > 0 || a.routed.y != nullptr);
+    const float fs = shared_factor(a.routed, n);
     float ss = 0.f;
     for (int c = threadIdx.x * V; c < d; c += blockDim.x * V) {
         Few<V> x = few<V>(r + c);
@@ -89,23 +47,8 @@ __global__ void __launch_bounds__(512) sum_norm_kernel(const SumNorm a) {
 #pragma unroll
                 for (int k = 0; k < V; ++k) x.v[k] = fmaf(a.coef[i], t.v[k], x.v[k]);
             }
-        if (a.y) {
-            Few<V> sum;
-#pragma unroll
-            for (int k = 0; k < V; ++k) sum.v[k] = 0.f;
-            for (int j = 0; j < a.top; ++j) {
-                const int p = a.place[n * a.top + j];
-                if (p < 0) continue;
-                const float w = a.weights[n * a.top + j];
-                const Few<V> t = few<V>(a.y + (int64_t)p * d + c);
-#pragma unroll
-                for (int k = 0; k < V; ++k) sum.v[k] = fmaf(w, t.v[k], sum.v[k]);
-            }
-            if (a.shared) {
-                const Few<V> t = few<V>(reinterpret_cast<const T*>(a.shared) + n * d + c);
-#pragma unroll
-                for (int k = 0; k < V; ++k) sum.v[k] = fmaf(fs, t.v[k], sum.v[k]);
-            }
+        if (a.routed.y) {
+            const Few<V> sum = routed_sum<T, V>(a.routed, n, d, c, fs);
 #pragma unroll
             for (int k = 0; k < V; ++k) x.v[k] += sum.v[k];
         }
@@ -211,8 +154,7 @@ SLLM_EXPORT int sllm_sum_norm(float* resid, const void* const* terms, const floa
         a.coef[i] = coefs[i];
         bits |= (uintptr_t)terms[i];
     }
-    a.y = y; a.ids = ids; a.weights = weights; a.place = place; a.top = top;
-    a.shared = shared; a.sg = sg; a.ldsg = ldsg;
+    a.routed = RoutedRows{y, ids, weights, place, top, shared, sg, ldsg};
     a.gA = gA; a.gB = gB; a.eps = eps; a.outA = outA; a.outB = outB;
     a.out_rows = out_rows; a.d = d;
     const bool vec = d % 4 == 0 && !(bits & 15);

@@ -16,7 +16,7 @@ import torch
 from ..config.spec import ModelSpec, PartSpec
 from ..kernels import ops
 from ..parts import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, POSITION_ENCODINGS, SIDE_INPUTS,
-                     STREAM_JOINS, TOKEN_EMBEDDINGS, TOKEN_MIXES, BuildContext, CacheView, KVSpec,
+                     STREAM_JOINS, STREAM_MIXES, TOKEN_EMBEDDINGS, TOKEN_MIXES, BuildContext, CacheView, KVSpec,
                      StateSpec, make)
 from ..parts.linear import Linear
 from ..parts.stream import Current, Normed, StreamSink
@@ -30,7 +30,8 @@ def _spec_key(spec: PartSpec):
 #: kind of part (a value of a block's ``ROLES``) -> (registry, name used in error messages)
 PART_KINDS = {"mixer": (MIXERS, "mixer"), "feed_forward": (FEED_FORWARDS, "feed-forward"),
               "norm": (NORMS, "norm"), "position": (POSITION_ENCODINGS, "position encoding"),
-              "side": (SIDE_INPUTS, "side input"), "token_mix": (TOKEN_MIXES, "token mix")}
+              "side": (SIDE_INPUTS, "side input"), "token_mix": (TOKEN_MIXES, "token mix"),
+              "stream_mix": (STREAM_MIXES, "stream mix")}
 
 
 def _tensor_name(prefix: str, name: str) -> str:
@@ -117,6 +118,17 @@ class DecoderModel:
             entry = nxt.entry() if nxt is not None and hasattr(nxt, "entry") else None
             self._next_entry.append(entry if getattr(block, "takes_next_entry", False) else None)
         self.final_norm = make(NORMS, "norm", spec.final_norm)
+        if spec.streams is not None:
+            if spec.embed_norm is not None or spec.token_embedding is not None or spec.joins \
+                    or spec.position_sinusoid_base > 0:
+                raise ValueError("a stream of several parts beside a norm after the embedding, a "
+                                 "token embedding, joins or sinusoidal positions is not built")
+            for norm in [self.final_norm] + [p for b in self.blocks for r, p in b.parts.items()
+                                             if b.ROLES[r] == "norm"]:
+                if not getattr(norm, "takes_streams", False):
+                    raise ValueError("a stream of several parts needs norms that read one "
+                                     "(takes_streams)")
+                norm.on_streams = True
         self._named_parts.append((spec.final_norm_name, self.final_norm))
         # a norm between the embedding and the first layer, for designs that have one
         self.embed_norm = None
@@ -139,7 +151,7 @@ class DecoderModel:
         entry = first.entry() if first is not None and hasattr(first, "entry") else None
         self._first_entry = entry if (entry is not None and getattr(entry[0], "deferrable", False)
                                       and hasattr(entry[1], "accepts_normed")
-                                      and spec.embed_norm is None
+                                      and spec.embed_norm is None and spec.streams is None
                                       and spec.token_embedding is None) else None
         # the last run may prepare the final norm for the output matrix in steps that want the
         # logits of every token in order (decode steps), where no rows are gathered in between
@@ -280,6 +292,8 @@ class DecoderModel:
         said = [jobs for jobs in said if jobs is not None]
         if not said:
             return None
+        # (parts that leave the choice to the others, but reach a library in long steps)
+        said += [p.long_step_jobs(dtype) for p in self.all_parts() if hasattr(p, "long_step_jobs")]
         names = ["sllm_elementwise", "sllm_sampling", "sllm_stream_ops"]
         names += ["sllm_gemm_simt"] if dtype == torch.float32 else ["sllm_gemv_mma", "sllm_gemv_tma"]
         return [ops.core_job(n) for n in names] + [job for jobs in said for job in jobs]
@@ -331,8 +345,9 @@ class DecoderModel:
         """Run the batch's tokens from the cache; returns logits [n_out, vocab] in 32-bit, or
         None when no logits are wanted."""
         s = self.spec
-        resid = torch.empty((batch.n_tokens, s.hidden_size), dtype=torch.float32,
-                            device=self.ctx.device)
+        shape = (batch.n_tokens, s.hidden_size) if s.streams is None else \
+            (batch.n_tokens, s.streams, s.hidden_size)
+        resid = torch.empty(shape, dtype=torch.float32, device=self.ctx.device)
         pending = self._embed(batch, resid, cache)
         if self.embed_norm is not None:
             if pending is not None:

@@ -49,6 +49,8 @@ EXTRA_LIBRARIES: dict[str, tuple[tuple[str, ...], tuple[str, ...]]] = {
     "sllm_norm_rope_cache": (("norm_rope_cache.cu",), ()),
     "sllm_gated_scan": (("gated_scan.cu",), ()),
     "sllm_sum_norm": (("sum_norm.cu",), ()),
+    "sllm_streams": (("streams.cu",), ()),
+    "sllm_channel_scan": (("channel_scan.cu",), ()),
 }
 
 
@@ -202,7 +204,7 @@ def _code(dtype: torch.dtype) -> int:
 def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor,
           pending: torch.Tensor | None = None, scale: float = 1.0) -> torch.Tensor:
     """out[n] = table[ids[n]] widened to 32-bit, times ``scale`` (an architecture's embedding
-    multiplier).  ids int32 [N]; table [V, d]; out f32 [N, d].
+    multiplier).  ids int32 [N]; table [V, d]; out f32 [N, d], or [N, S, d] for S equal parts.
     An id ``-1 - j`` stands for ``pending[j]`` (int32, on the device): a token that an earlier
     kernel of the stream chose and the host has not read yet."""
     _need(ids, torch.int32, "ids")
@@ -211,11 +213,13 @@ def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor,
     _need(table, None, "table")
     _need(out, torch.float32, "out")
     n, d = ids.numel(), table.shape[1]
-    if out.shape != (n, d):
-        raise KernelError(f"out must be [{n}, {d}], got {list(out.shape)}")
+    copies = out.shape[1] if out.dim() == 3 else 1
+    if out.shape not in ((n, d), (n, copies, d)):
+        raise KernelError(f"out must be [{n}, {d}] or [{n}, parts, {d}], got {list(out.shape)}")
     _check(_core("sllm_elementwise").sllm_embed(
         _ptr(ids), _ptr(pending) if pending is not None else c_void_p(0), _ptr(table), _ptr(out),
-        c_int(n), c_int(d), c_int(_code(table.dtype)), c_float(scale), _stream()), "embed")
+        c_int(n), c_int(d), c_int(_code(table.dtype)), c_float(scale), c_int(copies), _stream()),
+        "embed")
     return out
 
 
@@ -362,6 +366,24 @@ def gemv_mma(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bool =
         _ptr(x), _ptr(w), _ptr(out), c_int(m), c_int(n), c_int(k), c_int64(x.stride(0)),
         c_int64(w.stride(0)), c_int64(out.stride(0)), c_int(_gate_code(swiglu, activation)),
         c_int(_code(out.dtype)), *_gate_params(activation), _stream()), "gemv_mma")
+    return out
+
+
+def gemv_mma_groups(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """``out[g] = x[g] @ w[g]^T`` for a few products of equal sizes in one launch: ``x`` [G, M, K]
+    and ``w`` [G, N, K] bfloat16 with M <= 8 and rows of whole 16 bytes, ``out`` [G, M, N] (float32
+    or bfloat16; any strides with contiguous rows)."""
+    _need(x, torch.bfloat16, "x", contiguous=False)
+    _need(w, torch.bfloat16, "w", contiguous=False)
+    _need(out, None, "out", contiguous=False)
+    (g, m, k), (g2, n, k2) = x.shape, w.shape
+    if g != g2 or k != k2 or out.shape != (g, m, n) or x.stride(2) != 1 or w.stride(2) != 1 \
+            or out.stride(2) != 1:
+        raise KernelError("gemv_mma_groups shapes/strides")
+    _check(_core("sllm_gemv_mma").sllm_gemv_mma_groups(
+        _ptr(x), _ptr(w), _ptr(out), c_int(g), c_int(m), c_int(n), c_int(k), c_int64(x.stride(1)),
+        c_int64(w.stride(1)), c_int64(out.stride(1)), c_int64(x.stride(0)), c_int64(w.stride(0)),
+        c_int64(out.stride(0)), c_int(_code(out.dtype)), _stream()), "gemv_mma_groups")
     return out
 
 
@@ -1399,7 +1421,7 @@ MOE_PLAIN, MOE_GATED, MOE_SQRELU = 0, 1, 2
 
 def moe_route(logits: torch.Tensor, correction: torch.Tensor | None, token_row: torch.Tensor | None,
               n_real: int, n_groups: int, keep: int, top: int, tile_rows: int | None = None,
-              gather_from: torch.Tensor | None = None, flags: int = 0):
+              gather_from: torch.Tensor | None = None, flags: int = 0, scale: float = 1.0):
     """Route every token of ``logits`` (float32 [N, outputs], may be a column slice) and sort the
     (token, choice) pairs by expert (csrc/moe.cu).  Returns ``(ids [N, top], weights [N, top],
     pair_token [N * top], pair_place [N * top], meta, max_tiles, rows)``; ``meta`` is the tile list
@@ -1409,7 +1431,8 @@ def moe_route(logits: torch.Tensor, correction: torch.Tensor | None, token_row: 
     where one CTA does everything in one launch), else None (:func:`moe_gather_rows` makes it).
     ``flags``: ``MOE_SIGMOID`` scores are ``sigmoid(z)`` instead of a softmax over the outputs;
     ``MOE_GROUP_TOP2`` a group's score is the sum of its two largest choice scores instead of its
-    largest; ``MOE_RAW_WEIGHTS`` the weights are the chosen scores, not divided by their sum."""
+    largest; ``MOE_RAW_WEIGHTS`` the weights are the chosen scores, not divided by their sum.
+    ``scale`` multiplies the weights."""
     _need(logits, torch.float32, "logits", contiguous=False)
     n, n_total = logits.shape
     if logits.stride(1) != 1:
@@ -1446,7 +1469,7 @@ def moe_route(logits: torch.Tensor, correction: torch.Tensor | None, token_row: 
             _ptr(meta), c_int(max_tiles), c_int(tile_rows), _ptr(pair_token), _ptr(pair_place),
             _ptr(gather_from), c_int64(gather_from.stride(0) if gather_from is not None else 0),
             c_int(gather_from.shape[1] if gather_from is not None else 0), _ptr(rows),
-            c_int(flags), _stream()), "moe_route_small")
+            c_int(flags), c_float(scale), _stream()), "moe_route_small")
         return ids, weights, pair_token, pair_place, meta, max_tiles, rows
     # one zero fill: the experts' counters (with the offsets, cursors and tile list behind them)
     # and the places' tokens (places that no pair takes name token 0)
@@ -1458,7 +1481,7 @@ def moe_route(logits: torch.Tensor, correction: torch.Tensor | None, token_row: 
         c_int(n_total), c_int(n_real),
         c_int(n_groups), c_int(keep), c_int(top), _ptr(ids), _ptr(weights), _ptr(work),
         c_int(max_tiles), c_int(tile_rows), _ptr(pair_token), _ptr(pair_place), c_int(flags),
-        _stream()), "moe_route")
+        c_float(scale), _stream()), "moe_route")
     meta = work[3 * n_real + 1:]
     return ids, weights, pair_token, pair_place, meta, max_tiles, None
 
@@ -1649,13 +1672,18 @@ def _delta_rule_channels(act, ab, state, row_start, row_slot, out, n_rows, n_hea
 
 def lowrank_expand(pre: torch.Tensor, col0: int, w2t: torch.Tensor, out: torch.Tensor,
                    bias: torch.Tensor | None = None, rate_log: torch.Tensor | None = None,
-                   per_rate: int = 0, also: tuple | None = None) -> torch.Tensor:
+                   per_rate: int = 0, also: tuple | None = None, log_decay: str | None = None,
+                   rate: float = 1.0, tanh_in: bool = False) -> torch.Tensor:
     """The second product of a low-rank pair in 32-bit (csrc/recurrent_ops.cu): ``pre`` float32
     [N, *] holds the hidden values in columns ``[col0, col0 + R)``, ``w2t`` float32 [R, C];
     ``out`` [N, C] (float32 or bfloat16) gets ``bias + hidden w2t``, or, with ``rate_log``
     (float32 [C / per_rate]), ``-exp(rate_log[c // per_rate]) * softplus(bias + hidden w2t)``:
     the logarithm of a decay per channel.  ``also = (col0, w2t, out)``: a second plain product of
-    the same ``pre`` in the same launch."""
+    the same ``pre`` in the same launch.  ``log_decay``: with z the sum, "sigmoid" stores ``rate *
+    log sigmoid(z)``, "exp" stores ``-exp(z)``, both at least -88 (the logarithm of a decay that
+    leaves nothing).  ``tanh_in``: the hidden values pass a tanh first."""
+    if log_decay not in (None, "sigmoid", "exp") or (log_decay and rate_log is not None):
+        raise KernelError(f"lowrank_expand: unknown log_decay {log_decay!r}")
     _need(pre, torch.float32, "pre", contiguous=False)
     n = pre.shape[0]
     if pre.stride(1) != 1:
@@ -1678,12 +1706,14 @@ def lowrank_expand(pre: torch.Tensor, col0: int, w2t: torch.Tensor, out: torch.T
             if per < 1 or c % per or rl.numel() != c // per:
                 raise KernelError("lowrank_expand: one rate per `per_rate` channels")
     k = len(jobs)
+    modes = [1 if rate_log is not None else {None: 0, "sigmoid": 2, "exp": 3}[log_decay], 0][:k]
     ints = lambda vals: (c_int * k)(*vals)  # noqa: E731
     ptrs = lambda ts: (c_void_p * k)(*[None if t is None else t.data_ptr() for t in ts])  # noqa: E731
     _check(_core("sllm_recurrent_ops").sllm_lowrank_expand(
         _ptr(pre), c_int64(pre.stride(0)), c_int(k), ints([j[0] for j in jobs]),
         ptrs([j[1] for j in jobs]), ptrs([j[3] for j in jobs]), ptrs([j[4] for j in jobs]),
-        ints([j[5] for j in jobs]), ints([int(j[4] is not None) for j in jobs]),
+        ints([j[5] for j in jobs]), (c_float * k)(*([float(rate), 1.0][:k])),
+        ints([int(tanh_in), 0][:k]), ints(modes),
         ptrs([j[2] for j in jobs]), ints([_code(j[2].dtype) for j in jobs]),
         ints([j[1].shape[1] for j in jobs]), ints([j[1].shape[0] for j in jobs]), c_int(n),
         _stream()), "lowrank_expand")
@@ -1875,16 +1905,17 @@ LAYERNORM_MAX_TERMS = 4
 
 
 def add_layernorm(resid: torch.Tensor, terms: Sequence[tuple[torch.Tensor, float]],
-                  weight: torch.Tensor, bias: torch.Tensor, eps: float, out: torch.Tensor,
+                  weight: torch.Tensor, bias: torch.Tensor | None, eps: float, out: torch.Tensor,
                   out_rows: torch.Tensor | None = None) -> torch.Tensor:
     """``x = resid + sum(coef * term)`` in 32-bit, then ``out = (x - mean) / sqrt(var + eps) *
-    weight + bias`` (csrc/layer_norm.cu).  Without ``out_rows`` the stream ``resid`` is updated
+    weight + bias`` (csrc/layer_norm.cu; ``bias`` None: no offset).  Without ``out_rows`` the stream ``resid`` is updated
     in place and every token is normed; with ``out_rows`` (int32) only those tokens are, and the
     stream is not written.  ``out`` float32 or bfloat16; it may be ``resid`` itself when there
     are no terms (the stream normed in place)."""
     _need(resid, torch.float32, "resid")
     _need(weight, torch.float32, "weight")
-    _need(bias, torch.float32, "bias")
+    if bias is not None:
+        _need(bias, torch.float32, "bias")
     _need(out, None, "out")
     n, d = resid.shape
     if len(terms) > LAYERNORM_MAX_TERMS:
@@ -1902,7 +1933,7 @@ def add_layernorm(resid: torch.Tensor, terms: Sequence[tuple[torch.Tensor, float
     n_out = n if out_rows is None else out_rows.numel()
     if out_rows is not None:
         _need(out_rows, torch.int32, "out_rows")
-    if weight.numel() != d or bias.numel() != d or out.shape != (n_out, d):
+    if weight.numel() != d or (bias is not None and bias.numel() != d) or out.shape != (n_out, d):
         raise KernelError("add_layernorm shapes")
     ptrs = (c_void_p * LAYERNORM_MAX_TERMS)(*[t.data_ptr() for t, _ in terms])
     coefs = (c_float * LAYERNORM_MAX_TERMS)(*[float(c) for _, c in terms])
@@ -1964,6 +1995,32 @@ def norm_rope_kv_write(x: torch.Tensor, positions: torch.Tensor, token_row: torc
 SUM_NORM_MAX_TERMS = 4
 
 
+def _routed_args(routed, n: int, d: int, dtype: torch.dtype, what: str) -> tuple:
+    """A routed sum (an object with the fields of
+    :class:`scratch_llm_b200.parts.stream.RoutedSum`, or None) as launcher arguments."""
+    y = ids = weights = place = shared = gate = None
+    top = 0
+    if routed is not None:
+        y, ids, weights, place = routed.y, routed.ids, routed.weights, routed.place
+        shared, gate, top = routed.shared, routed.gate, routed.ids.shape[1]
+        _need(y, torch.float32, "y")
+        _need(ids, torch.int32, "ids")
+        _need(weights, torch.float32, "weights")
+        _need(place, torch.int32, "place")
+        if y.shape[1] != d or ids.shape[0] != n or place.numel() != n * top:
+            raise KernelError(f"{what}: the routed sum's shapes")
+        if shared is not None:
+            _need(shared, dtype, "shared")
+            if shared.shape != (n, d):
+                raise KernelError(f"{what}: the shared expert's output has the stream's shape")
+        if gate is not None:
+            _need(gate, torch.float32, "gate", contiguous=False)
+            if shared is None or gate.shape != (n, 1):
+                raise KernelError(f"{what}: a shared expert's gate has one number per token")
+    return (_ptr(y), _ptr(ids), _ptr(weights), _ptr(place), c_int(top), _ptr(shared), _ptr(gate),
+            c_int64(gate.stride(0) if gate is not None else 0))
+
+
 def sum_norm(resid: torch.Tensor, terms: Sequence[tuple[torch.Tensor, float]], gain: torch.Tensor,
              eps: float, out: torch.Tensor, gain_b: torch.Tensor | None = None,
              out_b: torch.Tensor | None = None, routed=None,
@@ -1995,33 +2052,62 @@ def sum_norm(resid: torch.Tensor, terms: Sequence[tuple[torch.Tensor, float]], g
             _need(o, out.dtype, "out")
             if w.numel() != d or o.shape != (n_out, d):
                 raise KernelError("sum_norm shapes")
-    y = ids = weights = place = shared = gate = None
-    top = 0
-    if routed is not None:
-        y, ids, weights, place = routed.y, routed.ids, routed.weights, routed.place
-        shared, gate, top = routed.shared, routed.gate, routed.ids.shape[1]
-        _need(y, torch.float32, "y")
-        _need(ids, torch.int32, "ids")
-        _need(weights, torch.float32, "weights")
-        _need(place, torch.int32, "place")
-        if y.shape[1] != d or ids.shape[0] != n or place.numel() != n * top:
-            raise KernelError("sum_norm: the routed sum's shapes")
-        if shared is not None:
-            _need(shared, out.dtype, "shared")
-            if shared.shape != (n, d):
-                raise KernelError("sum_norm: the shared expert's output has the stream's shape")
-        if gate is not None:
-            _need(gate, torch.float32, "gate", contiguous=False)
-            if shared is None or gate.shape != (n, 1):
-                raise KernelError("sum_norm: a shared expert's gate has one number per token")
+    routed_args = _routed_args(routed, n, d, out.dtype, "sum_norm")
     ptrs = (c_void_p * SUM_NORM_MAX_TERMS)(*[t.data_ptr() for t, _ in terms])
     coefs = (c_float * SUM_NORM_MAX_TERMS)(*[float(c) for _, c in terms])
     _check(_core("sllm_sum_norm").sllm_sum_norm(
-        _ptr(resid), ptrs, coefs, c_int(len(terms)), _ptr(y), _ptr(ids), _ptr(weights),
-        _ptr(place), c_int(top), _ptr(shared), _ptr(gate),
-        c_int64(gate.stride(0) if gate is not None else 0), _ptr(gain), _ptr(gain_b),
+        _ptr(resid), ptrs, coefs, c_int(len(terms)), *routed_args, _ptr(gain), _ptr(gain_b),
         c_float(eps), _ptr(out), _ptr(out_b), _ptr(out_rows), c_int(n_out), c_int(d),
         c_int(_code(out.dtype)), _stream()), "sum_norm")
+    return out
+
+
+STREAMS_MAX = 16
+STREAMS_MAX_TERMS = 4
+
+
+def streams_norm(parts: torch.Tensor, read: torch.Tensor | None, gain: torch.Tensor,
+                 bias: torch.Tensor | None, eps: float, rms: bool, out: torch.Tensor,
+                 mix: torch.Tensor | None = None, to: torch.Tensor | None = None,
+                 terms: Sequence[tuple[torch.Tensor, float]] = (), routed=None,
+                 out_rows: torch.Tensor | None = None) -> torch.Tensor:
+    """A residual stream of several parts ``parts`` float32 [N, S, d] (csrc/streams.cu): with
+    ``mix`` (float32 [S, S], [from, to]) and ``to`` (float32 [S]) first ``x_t <- sum_s mix[s, t]
+    x_s + to[t] y``, where ``y = sum(coef * term) + routed`` (as in :func:`sum_norm`); then ``out =
+    norm(sum_s read[s] x_s)`` (``read`` None: the plain sum), a layer norm (``bias`` may be None)
+    or, with ``rms``, an RMS norm.  Without ``out_rows`` the parts are updated in place; with
+    ``out_rows`` (int32) only those tokens are normed, and the parts are not written."""
+    _need(parts, torch.float32, "parts")
+    _need(gain, torch.float32, "gain")
+    _need(out, None, "out")
+    if parts.dim() != 3:
+        raise KernelError("streams_norm: the parts are [tokens, parts, width]")
+    n, s, d = parts.shape
+    n_out = n
+    if out_rows is not None:
+        _need(out_rows, torch.int32, "out_rows")
+        n_out = out_rows.numel()
+    if (mix is None) != (to is None) or (mix is None and (terms or routed is not None)):
+        raise KernelError("streams_norm: an update has both mixing weights")
+    for t, name, size in ((mix, "mix", s * s), (to, "to", s), (read, "read", s), (bias, "bias", d),
+                          (gain, "gain", d)):
+        if t is not None:
+            _need(t, torch.float32, name)
+            if t.numel() != size:
+                raise KernelError(f"streams_norm: {name} must have {size} entries")
+    if not 1 <= s <= STREAMS_MAX or len(terms) > STREAMS_MAX_TERMS or out.shape != (n_out, d):
+        raise KernelError("streams_norm shapes")
+    for t, _ in terms:
+        _need(t, out.dtype, "term")
+        if t.shape != (n, d):
+            raise KernelError("streams_norm: a term must have a part's shape")
+    ptrs = (c_void_p * STREAMS_MAX_TERMS)(*[t.data_ptr() for t, _ in terms])
+    coefs = (c_float * STREAMS_MAX_TERMS)(*[float(c) for _, c in terms])
+    _check(_core("sllm_streams").sllm_streams_norm(
+        _ptr(parts), c_int(s), _ptr(mix), _ptr(to), ptrs, coefs, c_int(len(terms)),
+        *_routed_args(routed, n, d, out.dtype, "streams_norm"), _ptr(read), _ptr(gain), _ptr(bias),
+        c_float(eps), c_int(int(rms)), _ptr(out), _ptr(out_rows), c_int(n_out), c_int(d),
+        c_int(_code(out.dtype)), _stream()), "streams_norm")
     return out
 
 
@@ -2062,11 +2148,12 @@ GATED_SCAN_MIN_CHUNKED = 64
 
 
 def gated_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: torch.Tensor,
-               weight: torch.Tensor, state: torch.Tensor, row_start: torch.Tensor,
+               weight: torch.Tensor | None, state: torch.Tensor, row_start: torch.Tensor,
                row_slot: torch.Tensor, out: torch.Tensor, n_rows: int, n_groups: int, key_dim: int,
                value_dim: int, longest: int, ones_out: torch.Tensor | None = None,
                skip: torch.Tensor | None = None, scale: float = 1.0,
-               min_chunked: int | None = None, shortest: int = 1) -> torch.Tensor:
+               min_chunked: int | None = None, shortest: int = 1,
+               silu: bool = False) -> torch.Tensor:
     """The recurrence ``S <- exp(log_decay) S + weight k v^T``, ``out = scale S^T q + skip v`` over
     the packed batch (csrc/gated_scan.cu): ``q``, ``k`` [N, G * key_dim] and ``v`` [N, H *
     value_dim] (may be column slices; head h reads group ``h // (H / G)``), ``log_decay`` (at
@@ -2076,20 +2163,24 @@ def gated_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: tor
     always 1 (a normaliser), whose read-out (times ``scale``) goes there.  ``longest``: the most
     tokens a row brings (an upper bound).  ``min_chunked``: rows of at least so many tokens run in
     chunks on the tensor cores (bfloat16, sizes in multiples of 16 and 8; 0: never).
-    ``shortest``: the fewest tokens a row brings (a lower bound)."""
+    ``shortest``: the fewest tokens a row brings (a lower bound).  A ``log_decay`` of shape [H] is
+    every token's, ``weight`` None is 1.  ``silu``: q, k and v pass a silu first (only without
+    chunks; a step with chunks takes them from :func:`silu_columns`)."""
     _need(q, None, "q", contiguous=False)
     _need(k, q.dtype, "k", contiguous=False)
     _need(v, q.dtype, "v", contiguous=False)
     for t, name in ((log_decay, "log_decay"), (weight, "weight"), (state, "state"), (out, "out")):
-        _need(t, torch.float32, name)
+        if t is not None:
+            _need(t, torch.float32, name)
     _need(row_start, torch.int32, "row_start")
     _need(row_slot, torch.int32, "row_slot")
-    n, n_heads = log_decay.shape
+    n, n_heads = q.shape[0], log_decay.shape[-1]
     ones = int(ones_out is not None)
     for t, width in ((q, n_groups * key_dim), (k, n_groups * key_dim), (v, n_heads * value_dim)):
         if t.shape != (n, width) or t.stride(1) != 1:
             raise KernelError("gated_scan: q, k and v are [tokens, groups or heads * size]")
-    if n_heads % n_groups or weight.shape != (n, n_heads) or out.shape != (n, n_heads * value_dim) \
+    if n_heads % n_groups or log_decay.shape not in ((n_heads,), (n, n_heads)) or \
+            (weight is not None and weight.shape != (n, n_heads)) or out.shape != (n, n_heads * value_dim) \
             or state.shape[1:] != (n_heads, value_dim + ones, key_dim):
         raise KernelError("gated_scan shapes")
     if not 1 <= key_dim <= GATED_SCAN_MAX_KEY_DIM:
@@ -2108,7 +2199,7 @@ def gated_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: tor
         min_chunked = GATED_SCAN_MIN_CHUNKED
     aligned = all(t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in (q, k, v))
     chunked = bool(min_chunked and longest >= min_chunked and q.dtype == torch.bfloat16 and aligned
-                   and lib.sllm_gated_scan_chunks_fit(c_int(key_dim), c_int(value_dim)))
+                   and not silu and lib.sllm_gated_scan_chunks_fit(c_int(key_dim), c_int(value_dim)))
     dS = decay = None
     if chunked:
         slots = n // int(lib.sllm_gated_scan_chunk()) + n_rows + 1
@@ -2117,14 +2208,101 @@ def gated_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: tor
         decay = torch.empty((slots, n_heads), dtype=torch.float32, device=q.device)
     _check(lib.sllm_gated_scan(
         _ptr(q), c_int64(q.stride(0)), _ptr(k), c_int64(k.stride(0)), _ptr(v),
-        c_int64(v.stride(0)), _ptr(log_decay), _ptr(weight), _ptr(state), _ptr(row_start),
-        _ptr(row_slot), _ptr(out), _ptr(ones_out), _ptr(skip), c_float(scale), c_int(n),
+        c_int64(v.stride(0)), _ptr(log_decay), _ptr(weight),
+        c_int64(n_heads if log_decay.dim() == 2 else 0), c_int(int(silu)), _ptr(state),
+        _ptr(row_start), _ptr(row_slot), _ptr(out), _ptr(ones_out), _ptr(skip), c_float(scale), c_int(n),
         c_int(n_rows), c_int(n_heads), c_int(n_groups), c_int(key_dim), c_int(value_dim),
         c_int(ones), c_int(int(chunked)), c_int(min_chunked), c_int(shortest), c_int(longest),
         _ptr(dS),
         _ptr(decay), c_int(_code(q.dtype)), _stream()),
         "gated_scan_chunked" if chunked else "gated_scan")
     return out
+
+
+def channel_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: torch.Tensor,
+                 state: torch.Tensor, row_start: torch.Tensor, row_slot: torch.Tensor,
+                 out: torch.Tensor, n_rows: int, n_heads: int, key_dim: int, value_dim: int,
+                 longest: int, bonus: torch.Tensor | None = None, scale: float = 1.0,
+                 min_chunked: int | None = None, shortest: int = 1) -> torch.Tensor:
+    """A recurrence with one decay per key channel over the packed batch (csrc/channel_scan.cu):
+    ``S <- diag(exp(log_decay)) S + k v^T``, ``out = scale S^T q`` with the new state, or, with
+    ``bonus`` u (float32 [H * key_dim]), ``out = scale (S_old + diag(u) k v^T)^T q``.  ``q``, ``k``
+    [N, H * key_dim] and ``v`` [N, H * value_dim] may be column slices; ``log_decay`` (at most 0)
+    float32 [N, H * key_dim]; ``state`` float32 [slots, H, value_dim, key_dim] is read and written
+    at the rows' slots.  ``longest`` / ``shortest``: bounds of the tokens a row brings.
+    ``min_chunked``: rows of at least so many tokens run in chunks (0: never)."""
+    _need(q, None, "q", contiguous=False)
+    _need(k, q.dtype, "k", contiguous=False)
+    _need(v, q.dtype, "v", contiguous=False)
+    for t, name in ((log_decay, "log_decay"), (state, "state"), (out, "out"), (bonus, "bonus")):
+        if t is not None:
+            _need(t, torch.float32, name)
+    _need(row_start, torch.int32, "row_start")
+    _need(row_slot, torch.int32, "row_slot")
+    n, hk, hv = q.shape[0], n_heads * key_dim, n_heads * value_dim
+    for t, width in ((q, hk), (k, hk), (v, hv)):
+        if t.shape != (n, width) or t.stride(1) != 1:
+            raise KernelError("channel_scan: q, k and v are [tokens, heads * size]")
+    if log_decay.shape != (n, hk) or out.shape != (n, hv) or \
+            state.shape[1:] != (n_heads, value_dim, key_dim) or \
+            (bonus is not None and bonus.numel() != hk):
+        raise KernelError("channel_scan shapes")
+    if not 1 <= key_dim <= GATED_SCAN_MAX_KEY_DIM:
+        raise KernelError(f"channel_scan takes key sizes up to {GATED_SCAN_MAX_KEY_DIM}, got "
+                          f"{key_dim}")
+    lib = _core("sllm_channel_scan")
+    if min_chunked is None:
+        min_chunked = GATED_SCAN_MIN_CHUNKED
+    chunked = bool(min_chunked and longest >= min_chunked)
+    dS = decay = weights = None
+    if chunked:
+        tc = int(lib.sllm_channel_scan_chunk())
+        slots = n // tc + n_rows + 1
+        make = lambda *shape: torch.empty(shape, dtype=torch.float32, device=q.device)  # noqa: E731
+        dS = make(slots, n_heads, value_dim, key_dim)
+        decay = make(slots, n_heads, key_dim)
+        weights = make(slots, n_heads, tc, tc)
+    _check(lib.sllm_channel_scan(
+        _ptr(q), c_int64(q.stride(0)), _ptr(k), c_int64(k.stride(0)), _ptr(v),
+        c_int64(v.stride(0)), _ptr(log_decay), _ptr(bonus), _ptr(state), _ptr(row_start),
+        _ptr(row_slot), _ptr(out), c_float(scale), c_int(n), c_int(n_rows), c_int(n_heads),
+        c_int(key_dim), c_int(value_dim), c_int(int(chunked)), c_int(min_chunked), c_int(shortest),
+        c_int(longest), _ptr(dS), _ptr(decay), _ptr(weights), c_int(_code(q.dtype)), _stream()),
+        "channel_scan_chunked" if chunked else "channel_scan")
+    return out
+
+
+def shift_mix(h: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, token_row: torch.Tensor,
+              row_start: torch.Tensor, row_slot: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """A token shift in front of M projections (csrc/recurrent_ops.cu): ``out[m] = h + (h_prev - h)
+    * mu[m]`` for ``h`` [N, d], ``mu`` float32 [M, d], ``out`` [M, N, d] in the dtype of ``h``.
+    ``state`` float32 [slots, d] carries each request's last h; it is read and written here."""
+    _need(h, None, "h", contiguous=False)
+    _need(out, h.dtype, "out")
+    _need(mu, torch.float32, "mu")
+    _need(state, torch.float32, "state")
+    for t, name in ((token_row, "token_row"), (row_start, "row_start"), (row_slot, "row_slot")):
+        _need(t, torch.int32, name)
+    n, d = h.shape
+    m = mu.shape[0]
+    if h.stride(1) != 1 or mu.shape != (m, d) or out.shape != (m, n, d) or state.shape[1:] != (d,):
+        raise KernelError("shift_mix shapes")
+    _check(_core("sllm_recurrent_ops").sllm_shift_mix(
+        _ptr(h), c_int64(h.stride(0)), _ptr(mu), c_int(m), _ptr(state), _ptr(token_row),
+        _ptr(row_start), _ptr(row_slot), _ptr(out), c_int(n), c_int(d), c_int(_code(h.dtype)),
+        _stream()), "shift_mix")
+    return out
+
+
+def silu_columns(x: torch.Tensor) -> torch.Tensor:
+    """``x <- silu(x)`` in place; ``x`` [N, C] may be a column slice (csrc/recurrent_ops.cu)."""
+    _need(x, None, "x", contiguous=False)
+    if x.dim() != 2 or x.stride(1) != 1:
+        raise KernelError("silu_columns: rows must be contiguous")
+    _check(_core("sllm_recurrent_ops").sllm_silu_columns(
+        _ptr(x), c_int64(x.stride(0)), c_int(x.shape[0]), c_int(x.shape[1]), c_int(_code(x.dtype)),
+        _stream()), "silu_columns")
+    return x
 
 
 def ssd_gates(pre: torch.Tensor, bias: torch.Tensor, a_log: torch.Tensor,
@@ -2174,9 +2352,11 @@ def memory_gates(pre: torch.Tensor, bias_i: torch.Tensor, bias_f: torch.Tensor, 
 
 
 def gate_part_norm(o: torch.Tensor, gate: torch.Tensor, gain: torch.Tensor, eps: float,
-                   parts: int, out: torch.Tensor) -> torch.Tensor:
-    """``y = o * silu(gate)``, then each of ``parts`` equal parts of a token's ``y`` over its own
-    root mean square (eps inside the root), times ``gain``: the gate comes before the norm.
+                   parts: int, out: torch.Tensor, gate_activation: str = "silu",
+                   gate_after: bool = False) -> torch.Tensor:
+    """``y = o * act(gate)``, then each of ``parts`` equal parts of a token's ``y`` over its own
+    root mean square (eps inside the root), times ``gain``: the gate comes before the norm.  With
+    ``gate_after`` the norm of ``o`` comes first, then the gate.
     ``o`` float32 [N, W], ``gate`` [N, W] (may be a column slice), ``gain`` float32 [W]."""
     _need(o, torch.float32, "o")
     _need(gate, out.dtype, "gate", contiguous=False)
@@ -2186,8 +2366,11 @@ def gate_part_norm(o: torch.Tensor, gate: torch.Tensor, gain: torch.Tensor, eps:
     if gate.shape != (n, w) or out.shape != (n, w) or gate.stride(1) != 1 or out.stride(1) != 1 \
             or gain.numel() != w or parts < 1 or w % parts:
         raise KernelError("gate_part_norm shapes")
+    if gate_activation not in ("silu", "sigmoid"):
+        raise KernelError(f"unknown gate activation {gate_activation!r}")
     _check(_core("sllm_recurrent_ops").sllm_gate_part_norm(
         _ptr(o), _ptr(gate), c_int64(gate.stride(0)), _ptr(gain), c_float(eps), _ptr(out),
-        c_int64(out.stride(0)), c_int(n), c_int(w), c_int(parts), c_int(_code(out.dtype)),
+        c_int64(out.stride(0)), c_int(n), c_int(w), c_int(parts),
+        c_int(int(gate_activation == "sigmoid")), c_int(int(gate_after)), c_int(_code(out.dtype)),
         _stream()), "gate_part_norm")
     return out

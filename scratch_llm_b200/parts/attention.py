@@ -14,7 +14,8 @@ cache's pages have one head size: with a ``value_dim``, or a head size that is n
 16, every head is padded with zero rows of its projection up to a common multiple of 16, which
 changes no score (zeros meet zeros) and no output (the output projection gets zero columns).
 In steps of single tokens the decode kernel adds the biases and turns the rotated part itself,
-as it does for the plain form.
+as it does for the plain form.  The concatenated heads may also be written into a slice of a
+buffer that a block or mixer multiplies by one joined output matrix (``out_segments``).
 """
 
 from __future__ import annotations
@@ -96,7 +97,7 @@ class GQAttention(Mixer):
         if dtype == torch.bfloat16 and self.head_dim <= ops.MMA_MAX_HEAD_DIM:
             jobs.append(ops.attention_mma_library(self.head_dim))
             if ops.attention_tc_supports(self.n_heads, self.n_kv_heads, self.head_dim, 16,
-                                         self.window):
+                                         self.window, biased=True):
                 jobs.append(ops.attention_tc_library(self.head_dim))
         else:
             jobs.append(ops.attention_library(self.head_dim))
@@ -146,8 +147,22 @@ class GQAttention(Mixer):
         out = self._attend(x, batch, cache, write, position)
         return self.o(out) if sink is None else sink.finish(self.o, out)
 
-    def _attend(self, x, batch, cache: CacheView, write: bool,
-                position: PositionEncoding) -> torch.Tensor:
+    # -- for a block or mixer that multiplies several branches' activations by one joined matrix
+
+    def out_segments(self):
+        """[(the output matrix [hidden, H * head_dim], its weight in the layer's sum)]."""
+        return [(self.o.weight, 1.0)]
+
+    def release_out(self) -> None:
+        self.o = None
+
+    def activations_into(self, x, batch, cache: CacheView, write: bool, position, outs) -> None:
+        self._attend(x, batch, cache, write, position, out=outs[0])
+
+    def _attend(self, x, batch, cache: CacheView, write: bool, position: PositionEncoding,
+                out: torch.Tensor | None = None) -> torch.Tensor:
+        """The concatenated heads' outputs [N, H * head_dim].  ``out``: where to put them (may be a
+        column slice; in a padded step it must hold zeros)."""
         H, G, hd = self.n_heads, self.n_kv_heads, self.head_dim
         qkv = self.qkv(x)
         if position.rotary_tables:
@@ -159,8 +174,9 @@ class GQAttention(Mixer):
             cos = sin = None
             interleaved = True
         # (padding tokens get no attention output: zeros, so that what follows stays finite)
-        out = (torch.zeros if batch.padded else torch.empty)(
-            (qkv.shape[0], H * hd), dtype=qkv.dtype, device=qkv.device)
+        if out is None:
+            out = (torch.zeros if batch.padded else torch.empty)(
+                (qkv.shape[0], H * hd), dtype=qkv.dtype, device=qkv.device)
         if (cos is not None and qkv.dtype == torch.bfloat16 and batch.n_multi == 0
                 and batch.n_single > 0 and H // G <= 16
                 and ops.attention_decode_fused_supported(hd)):
@@ -217,11 +233,13 @@ class GQAttention(Mixer):
         common = (q, cache.pages, cache.block_table, cache.page_size, batch.row_start,
                   batch.row_pos0, out)
         if batch.n_multi:
-            if ops.attention_tc_supports(H, G, hd, cache.page_size, self.window) \
-                    and batch.max_new_multi * (H // G) >= TC_MIN_PACKED_QUERIES:
-                # tcgen05 kernel: scores, probabilities and output in tensor memory
+            if ops.attention_tc_supports(H, G, hd, cache.page_size, self.window, biased=True) \
+                    and batch.max_new_multi * (H // G) >= TC_MIN_PACKED_QUERIES \
+                    and out.stride(0) % 8 == 0:
+                # tcgen05 kernel: scores, probabilities and output in tensor memory (with a
+                # window: its entry that skips key tiles behind it)
                 ops.attention_tc(*common, batch.multi_rows, batch.n_multi, batch.max_new_multi,
-                                 H, G, hd, self.scale)
+                                 H, G, hd, self.scale, self.window)
             else:
                 ops.attention_mma(*common, batch.multi_rows, batch.n_multi,
                                   batch.max_new_multi, H, G, hd, self.scale, self.window,

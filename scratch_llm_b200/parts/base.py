@@ -21,6 +21,8 @@ TokenEmbedding     ``embed(batch, table, resid, scale, state)``: the embedded to
                    beside their own vectors, into the stream
 StreamJoin         ``forward(resid, first) -> resid``: the stream joined with the embedding
                    output, before a run that the model's run order marks
+StreamMix          how a sublayer reads a stream of several parts and what its output does to them:
+                   ``read`` (the reading weights) and ``update(output) -> pending``
 Block              ``forward(resid, pending, batch, cache, write) -> pending``: the arrangement
                    of a layer's parts around the residual stream; its ``ROLES`` says which
                    parts it has (role -> kind of part), and it is built with one keyword
@@ -203,10 +205,22 @@ class StreamJoin(Part):
         raise NotImplementedError
 
 
+class StreamMix(Part):
+    """How a sublayer reads a residual stream of several parts (``ModelSpec.streams``; the stream
+    is then [N, parts, hidden]) and what its output does to them: ``read`` (float32 [parts]) goes
+    to the norm in front of the sublayer, ``update(output)`` is what the sublayer leaves pending
+    (:class:`~.stream.StreamUpdate`), which the next norm carries out."""
+
+    read: torch.Tensor | None = None
+
+    def update(self, value):
+        raise NotImplementedError
+
+
 class Block:
     """An arrangement of a layer's parts.  ``ROLES`` maps each role the arrangement has onto
     the kind of part that fills it: ``"mixer"``, ``"feed_forward"``, ``"norm"`` or
-    ``"position"``, ``"side"`` or ``"token_mix"`` (the registry the part's spec is looked up in).  The model builds the parts
+    ``"position"``, ``"side"``, ``"token_mix"`` or ``"stream_mix"`` (the registry the part's spec is looked up in).  The model builds the parts
     from the layer's specs and constructs the block with one keyword argument per role.  At most
     one role may be a mixer: it owns the layer's cache entry."""
 

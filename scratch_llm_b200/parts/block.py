@@ -292,3 +292,45 @@ class ParallelNormsBlock(Block):
         a = Terms.of(self.mixer.forward(h, batch, cache, write, self.position))
         f = self.feed_forward.forward(g, lazy=True) if self._lazy else self.feed_forward.forward(g)
         return a + Terms.of(f)
+
+
+@register_block("hyper_connected")
+class HyperConnectedBlock(Block):
+    """A pre-norm layer on a residual stream of several parts: each sublayer reads a weighted sum of
+    the parts, and its output goes to every part while the parts mix (a stream mix per sublayer,
+    :mod:`.hyper_connection`).  The feed-forward (with its norm and stream mix) is optional.
+    Nothing is added here: a sublayer's output is handed on (:class:`~.stream.StreamUpdate`), a
+    routed feed-forward's before it is added up, and the norm of whoever reads the parts next
+    carries the update out."""
+
+    ROLES = {"mixer": "mixer", "mixer_norm": "norm", "mixer_streams": "stream_mix",
+             "feed_forward": "feed_forward", "feed_forward_norm": "norm",
+             "feed_forward_streams": "stream_mix", "position": "position"}
+    OPTIONAL_ROLES = frozenset({"feed_forward", "feed_forward_norm", "feed_forward_streams"})
+    pad_safe = True   # the arrangement itself touches no token: its parts decide
+
+    def __init__(self, mixer: Mixer, mixer_norm: Norm, mixer_streams, position: PositionEncoding,
+                 feed_forward: FeedForward | None = None, feed_forward_norm: Norm | None = None,
+                 feed_forward_streams=None) -> None:
+        if len({feed_forward is None, feed_forward_norm is None,
+                feed_forward_streams is None}) != 1:
+            raise ValueError("a feed-forward comes with its norm and its stream mix")
+        for norm in (mixer_norm, feed_forward_norm):
+            if norm is not None and not getattr(norm, "takes_streams", False):
+                raise ValueError("a hyper_connected block needs norms that read a stream of several "
+                                 "parts (takes_streams)")
+        self.mixer, self.mixer_norm, self.mixer_streams = mixer, mixer_norm, mixer_streams
+        self.position = position
+        self.feed_forward, self.feed_forward_norm = feed_forward, feed_forward_norm
+        self.feed_forward_streams = feed_forward_streams
+        self._lazy = getattr(feed_forward, "hands_on_routed", False)
+
+    def forward(self, resid: torch.Tensor, pending, batch, cache: CacheView, write: bool):
+        h = self.mixer_norm.forward(resid, pending, read=self.mixer_streams.read)
+        pending = self.mixer_streams.update(
+            self.mixer.forward(h, batch, cache, write, self.position))
+        if self.feed_forward is None:
+            return pending
+        h = self.feed_forward_norm.forward(resid, pending, read=self.feed_forward_streams.read)
+        f = self.feed_forward.forward(h, lazy=True) if self._lazy else self.feed_forward.forward(h)
+        return self.feed_forward_streams.update(f)

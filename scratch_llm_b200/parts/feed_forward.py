@@ -25,6 +25,11 @@ class SwiGLU(FeedForward):
     def accepts_normed(self, n_tokens: int) -> bool:
         return self.gate_up is not None and self.gate_up.takes_normed(n_tokens, swiglu=True)
 
+    def long_step_jobs(self, dtype):
+        """What steps of many tokens reach, for models whose other parts list their libraries: the
+        fused tcgen05 product."""
+        return [ops.core_job("sllm_gemm_tcgen05")] if dtype == torch.bfloat16 else []
+
     def __init__(self, hidden_size: int, intermediate_size: int,
                  names: Mapping[str, str] | None = None, activation: str = "silu") -> None:
         """``activation``: what the gate passes through, "silu" or "gelu_tanh"."""

@@ -141,3 +141,29 @@ class Linear:
         if activation == "silu" and out.is_contiguous():
             return ops.swiglu(self(x), out)
         return ops.gated_act(self(x), out, activation)
+
+
+class GroupedLinear:
+    """A few products of equal sizes, each with an input of its own: ``y[g] = x[g] @ W[g].T`` for
+    ``W`` [G, out, in].  Steps of a few tokens: one launch of the streaming kernel for all groups;
+    longer ones: the library's batched product; 32-bit: the CUDA-core kernel, group by group."""
+
+    def __init__(self, weight: torch.Tensor) -> None:
+        if weight.dim() != 3 or not weight.is_contiguous():
+            raise ValueError("a GroupedLinear weight is a contiguous [groups, out, in] tensor")
+        self.weight = weight
+
+    def __call__(self, x: torch.Tensor) -> torch.Tensor:
+        w = self.weight
+        if x.dtype != w.dtype or x.dim() != 3 or x.shape[0] != w.shape[0]:
+            raise ValueError(f"GroupedLinear: input {x.dtype} {list(x.shape)}, weight {w.dtype} "
+                             f"{list(w.shape)}")
+        g, m = x.shape[:2]
+        if w.dtype == torch.float32 or (m <= SMALL_BATCH and w.shape[2] % 8 == 0):
+            out = torch.empty((g, m, w.shape[1]), dtype=w.dtype, device=x.device)
+            if w.dtype == torch.float32:
+                for i in range(g):
+                    ops.gemm_simt(x[i], w[i], out[i])
+                return out
+            return ops.gemv_mma_groups(x, w, out)
+        return torch.bmm(x, w.transpose(1, 2))

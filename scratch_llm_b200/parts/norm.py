@@ -15,7 +15,21 @@ from ..kernels import ops
 from ..weights.loader import ParamSpec
 from .base import BuildContext, Norm
 from .registry import register_norm
-from .stream import Current, Normed, Terms
+from .stream import Current, Normed, StreamUpdate, Terms
+
+
+def _norm_streams(resid: torch.Tensor, pending, out_rows, read, gain, bias, eps: float, rms: bool,
+                  dtype: torch.dtype) -> torch.Tensor:
+    """A norm of what a sublayer reads from a stream of several parts [N, parts, d], with the
+    pending update (None or a StreamUpdate) carried out in the same pass."""
+    if pending is not None and not isinstance(pending, StreamUpdate):
+        raise ValueError("a stream of several parts takes a StreamUpdate as what is pending")
+    n = resid.shape[0] if out_rows is None else out_rows.numel()
+    out = torch.empty((n, resid.shape[2]), dtype=dtype, device=resid.device)
+    update = {} if pending is None else {
+        "mix": pending.mix, "to": pending.to, "terms": pending.terms.items,
+        "routed": pending.terms.routed}
+    return ops.streams_norm(resid, read, gain, bias, eps, rms, out, out_rows=out_rows, **update)
 
 
 @register_norm("rmsnorm")
@@ -26,6 +40,7 @@ class RMSNorm(Norm):
     deferrable = True
     takes_terms = True    # forward() accepts a Terms as what is pending
     takes_routed = True   # ... and a routed feed-forward's output in it
+    takes_streams = True  # forward(..., read=) norms what is read from a stream of several parts
 
     def __init__(self, size: int, eps: float, name: str = "weight", offset: float = 0.0) -> None:
         """``name``: the gain's tensor name below the part's prefix; "" if the prefix itself is
@@ -45,7 +60,11 @@ class RMSNorm(Norm):
         self.dtype = ctx.dtype
 
     def forward(self, resid: torch.Tensor, delta: torch.Tensor | None,
-                out_rows: torch.Tensor | None = None):
+                out_rows: torch.Tensor | None = None, read: torch.Tensor | None = None):
+        """``read`` (float32 [parts]): how a stream of several parts is read; None: their sum."""
+        if resid.dim() == 3:
+            return _norm_streams(resid, delta, out_rows, read, self.weight, None, self.eps, True,
+                                 self.dtype)
         if isinstance(delta, Normed):
             # the product before this norm has already put its output into the stream and
             # prepared this norm: what is left is the tokens' factor, which the next product applies
@@ -175,16 +194,18 @@ class DynamicTanh(Norm):
 class LayerNorm(Norm):
     """``(x - mean) / sqrt(var + eps) * w + b`` with the variance as the mean of the squared
     deviations, all in 32-bit with one rounding at the end.  Tensors below the part's prefix: the
-    gain under ``name`` ("" = the prefix itself) and the offset under ``<name>.b``.
+    gain under ``name`` ("" = the prefix itself) and the offset under ``<name>.b`` (``bias=False``:
+    there is none).
 
     What is pending for the stream may be a tensor or a weighted sum of several
     (:class:`~.stream.Terms`): the kernel adds them in while it reads the stream."""
 
     pad_safe = True       # every token by itself
     takes_terms = True    # forward() accepts a Terms as what is pending
+    takes_streams = True  # forward(..., read=) norms what is read from a stream of several parts
 
-    def __init__(self, size: int, eps: float, name: str = "") -> None:
-        self.size, self.eps, self.name = size, float(eps), name
+    def __init__(self, size: int, eps: float, name: str = "", bias: bool = True) -> None:
+        self.size, self.eps, self.name, self.has_bias = size, float(eps), name, bool(bias)
         self.weight: torch.Tensor | None = None
         self.bias: torch.Tensor | None = None
         self.dtype = torch.float32
@@ -192,16 +213,22 @@ class LayerNorm(Norm):
     def _bias_name(self) -> str:
         return f"{self.name}.b" if self.name else "b"
 
+    #: set by a model whose stream has several parts: the norm then only runs in that form
+    on_streams = False
+
     def kernel_jobs(self, dtype: torch.dtype):
-        return [ops.core_job("sllm_layer_norm")]
+        return [ops.core_job("sllm_streams" if self.on_streams else "sllm_layer_norm")]
 
     def param_specs(self) -> dict[str, ParamSpec]:
-        return {self.name: ParamSpec((self.size,), "gain"),
-                self._bias_name(): ParamSpec((self.size,), "gain")}
+        specs = {self.name: ParamSpec((self.size,), "gain")}
+        if self.has_bias:
+            specs[self._bias_name()] = ParamSpec((self.size,), "gain")
+        return specs
 
     def load(self, tensors: Mapping[str, torch.Tensor], ctx: BuildContext) -> None:
         f32 = lambda t: t.to(device=ctx.device, dtype=torch.float32).contiguous()  # noqa: E731
-        self.weight, self.bias = f32(tensors[self.name]), f32(tensors[self._bias_name()])
+        self.weight = f32(tensors[self.name])
+        self.bias = f32(tensors[self._bias_name()]) if self.has_bias else None
         self.dtype = ctx.dtype
 
     @staticmethod
@@ -215,7 +242,12 @@ class LayerNorm(Norm):
                              "hand it over")
         return ((delta, 1.0),)
 
-    def forward(self, resid: torch.Tensor, delta=None, out_rows: torch.Tensor | None = None):
+    def forward(self, resid: torch.Tensor, delta=None, out_rows: torch.Tensor | None = None,
+                read: torch.Tensor | None = None):
+        """``read`` (float32 [parts]): how a stream of several parts is read; None: their sum."""
+        if resid.dim() == 3:
+            return _norm_streams(resid, delta, out_rows, read, self.weight, self.bias, self.eps,
+                                 False, self.dtype)
         n = resid.shape[0] if out_rows is None else out_rows.numel()
         out = torch.empty((n, self.size), dtype=self.dtype, device=resid.device)
         return ops.add_layernorm(resid, self._terms(delta), self.weight, self.bias, self.eps,

@@ -20,6 +20,11 @@ dims - 1)``, the ramp is ``r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1)`` a
 ``f_i / factor * r_i + f_i * (1 - r_i)``; cos and sin are both multiplied by
 ``yarn_magnitude * ln(factor) + 1``.
 
+``llama3`` (a mapping ``factor``, ``low``, ``high``, ``original``; the scaling of Llama 3.1): with a
+pair's wavelength ``l = 2 pi / f``, ``f`` stays where ``l < original / high``, becomes ``f / factor``
+where ``l > original / low``, and between the two is the blend ``(1 - s) f / factor + s f`` with
+``s = (original / l - low) / (high - low)``.
+
 ``none``: no position encoding (a mixer that needs none, or a test part).
 """
 
@@ -42,7 +47,8 @@ class Rotary(PositionEncoding):
     def __init__(self, head_dim: int, theta: float, max_position: int,
                  interleaved: bool = True, rot_dims: int | None = None,
                  scaling_factor: float = 1.0, yarn: Mapping[str, Any] | None = None,
-                 yarn_magnitude: float = 0.1) -> None:
+                 yarn_magnitude: float = 0.1,
+                 llama3: Mapping[str, Any] | None = None) -> None:
         if head_dim % 2:
             raise ValueError(f"rotary positions need an even head size, got {head_dim}")
         if rot_dims is not None and (rot_dims % 2 or not 2 <= rot_dims <= head_dim):
@@ -60,8 +66,30 @@ class Rotary(PositionEncoding):
             raise ValueError(f"yarn scaling needs positive factor, original, fast and slow, "
                              f"got {yarn!r}")
         self.yarn_magnitude = float(yarn_magnitude)
+        self.llama3 = None if llama3 is None else {k: float(llama3[k])
+                                                   for k in ("factor", "low", "high", "original")}
+        if self.llama3 is not None and not (self.llama3["factor"] > 0 and
+                                            0 < self.llama3["low"] <= self.llama3["high"] and
+                                            self.llama3["original"] > 0):
+            raise ValueError("llama3 scaling needs a positive factor and original and 0 < low <= "
+                             f"high, got {llama3!r}")
+        if self.llama3 is not None and self.yarn is not None:
+            raise ValueError("frequencies are scaled one way, not two")
         self.cos: torch.Tensor | None = None
         self.sin: torch.Tensor | None = None
+
+    def _scaled(self, f: float) -> float:
+        """A pair's frequency after the scaling of Llama 3.1 (if there is one)."""
+        c = self.llama3
+        if c is None:
+            return f
+        turns = c["original"] * f / (2.0 * math.pi)     # original / wavelength
+        if turns > c["high"]:
+            return f
+        if turns < c["low"]:
+            return f / c["factor"]
+        s = (turns - c["low"]) / (c["high"] - c["low"]) if c["high"] > c["low"] else 1.0
+        return (1.0 - s) * f / c["factor"] + s * f
 
     def tables(self) -> tuple[torch.Tensor, torch.Tensor]:
         """The table on the CPU in 32-bit: the reference's, or, with ``rot_dims`` or a scaling
@@ -85,9 +113,10 @@ class Rotary(PositionEncoding):
             freqs = torch.arange(self.max_position).float()[:, None] * inv_freq[None, :]
             mag = self.yarn_magnitude * math.log(y["factor"]) + 1.0
             return freqs.cos() * mag, freqs.sin() * mag
-        if self.rot_dims is not None or self.scaling_factor != 1.0:
+        if self.rot_dims is not None or self.scaling_factor != 1.0 or self.llama3 is not None:
             dims = self.rot_dims or self.head_dim
-            inv_freq = torch.tensor([self.theta ** (-2.0 * j / dims) / self.scaling_factor
+            inv_freq = torch.tensor([self._scaled(self.theta ** (-2.0 * j / dims)
+                                                  / self.scaling_factor)
                                      for j in range(dims // 2)], dtype=torch.float64).float()
             freqs = torch.arange(self.max_position).float()[:, None] * inv_freq[None, :]
             return freqs.cos(), freqs.sin()

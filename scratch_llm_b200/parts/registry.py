@@ -17,6 +17,7 @@ SIDE_INPUTS: dict[str, Callable[..., Any]] = {}
 TOKEN_MIXES: dict[str, Callable[..., Any]] = {}
 STREAM_JOINS: dict[str, Callable[..., Any]] = {}
 TOKEN_EMBEDDINGS: dict[str, Callable[..., Any]] = {}
+STREAM_MIXES: dict[str, Callable[..., Any]] = {}
 BLOCKS: dict[str, Callable[..., Any]] = {}
 
 
@@ -39,6 +40,7 @@ register_side_input = _register(SIDE_INPUTS, "side input")
 register_token_mix = _register(TOKEN_MIXES, "token mix")
 register_stream_join = _register(STREAM_JOINS, "stream join")
 register_token_embedding = _register(TOKEN_EMBEDDINGS, "token embedding")
+register_stream_mix = _register(STREAM_MIXES, "stream mix")
 register_block = _register(BLOCKS, "block")
 
 

@@ -21,7 +21,7 @@ chosen scores s themselves) and ``expert="sqrelu"`` (experts without a gate,
 ``W_down(relu(W_up x)^2)``, tensors ``e<i>.{up,down}``); ``correction=False`` (the choice is by the
 scores alone, there is no such tensor) and ``shared_gate=True`` (the shared expert's output is
 multiplied by ``sigmoid(w_sg . x)``, one number per token, tensor ``shared.sg``; its logit comes
-out of the router's product).  A softmax over all outputs whose chosen scores are divided by
+out of the router's product); ``weight_scale`` multiplies the weights.  A softmax over all outputs whose chosen scores are divided by
 their sum is the softmax over the chosen outputs' logits alone.
 
 A block and a norm that take it get the output before it is added up (``lazy=True``:
@@ -57,7 +57,7 @@ class RoutedExperts(FeedForward):
                  shared_size: int | None = None, score: str = "softmax",
                  group_score: str = "max", renormalize: bool = True,
                  expert: str = "gated_silu", correction: bool = True,
-                 shared_gate: bool = False) -> None:
+                 shared_gate: bool = False, weight_scale: float = 1.0) -> None:
         total = experts + identity
         if experts < 0 or identity < 0 or total < 1:
             raise ValueError("a router needs at least one output")
@@ -82,6 +82,7 @@ class RoutedExperts(FeedForward):
         self.groups, self.keep_groups = groups, keep_groups
         if shared_gate and shared_size is None:
             raise ValueError("a shared expert's gate needs a shared expert")
+        self.weight_scale = float(weight_scale)
         self.has_correction, self.shared_gate = bool(correction), bool(shared_gate)
         #: forward() takes lazy=: the output may be handed on before it is added up
         self.hands_on_routed = identity == 0 and experts > 0
@@ -156,7 +157,7 @@ class RoutedExperts(FeedForward):
         ids, weights, pair_token, pair_place, meta, max_tiles, rows = ops.moe_route(
             logits, self.correction, None, self.experts, self.groups, self.keep_groups, self.top,
             tile_rows=ops.MOE_TC_TILE_ROWS if tensor_cores else None,
-            gather_from=x if tensor_cores else None, flags=self.flags)
+            gather_from=x if tensor_cores else None, flags=self.flags, scale=self.weight_scale)
         pairs = n * self.top
         y = torch.empty((max(pairs, 1), d), dtype=torch.float32, device=x.device)
         if self.experts:

@@ -6,6 +6,10 @@ this mixer shares it out: paged keys and values for the side that wants them (at
 may), per-request state for each side that keeps some (the entry's state tensors are the left
 side's followed by the right side's).  Nothing is added here: the result is handed on as a
 weighted sum (:class:`~.stream.Terms`) for a block and a norm that take one.
+
+Where both sides end with a matrix product and one of them can scale its activations ahead of their
+rounding (``scale_activations``), the two products are one over the concatenated activations:
+``l W_l a_l + r W_r a_r = l [W_l | W_r] [a_l; (r / l) a_r]``, with the matrices as they are.
 """
 
 from __future__ import annotations
@@ -15,6 +19,7 @@ from typing import Any, Mapping
 import torch
 
 from .base import BuildContext, CacheView, KVSpec, Mixer, PositionEncoding
+from .linear import Linear
 from .registry import MIXERS, register_mixer
 from .stream import Terms
 
@@ -41,6 +46,12 @@ class SideBySide(Mixer):
         self.scales = (float(left_scale), float(right_scale))
         self.names = {"left": "left", "right": "right", **(names or {})}
         self.prefixes = (self.names["left"], self.names["right"])
+        #: the sides' output matrices side by side, once the weights are there: None = not tried yet,
+        #: False = they stay apart
+        self._joint = None
+        self._joint_scale = 1.0
+        self._widths: list[tuple[int, int]] = []     # per side: (first column, width)
+        self._zero_fill = False
         if sum(side.kv_spec() is not None for side in self.sides) > 1:
             raise ValueError("both sides want paged keys and values: a layer's cache entry has "
                              "one set of pages")
@@ -107,7 +118,48 @@ class SideBySide(Mixer):
                                    page_size=cache.page_size, state=state))
         return views
 
+    def _join_outputs(self) -> None:
+        """One output matrix for both sides, if they can (see above); the side that scales its
+        activations takes the quotient of the two weights, the other's goes to the sum."""
+        self._joint = False
+        segments = [side.out_segments() if hasattr(side, "out_segments") else None
+                    for side in self.sides]
+        if any(s is None or len(s) != 1 for s in segments):
+            return
+        scales = [scale * s[0][1] for scale, s in zip(self.scales, segments)]
+        fold = next((i for i, side in enumerate(self.sides) if hasattr(side, "scale_activations")
+                     and scales[1 - i] != 0.0), None)
+        if scales[0] != scales[1]:
+            if fold is None:
+                return
+            self.sides[fold].scale_activations(scales[fold] / scales[1 - fold])
+            self._joint_scale = scales[1 - fold]
+        else:
+            self._joint_scale = scales[0]
+        blocks, at = [], 0
+        for ((w, _),) in segments:
+            width = w.shape[1]
+            padded = -(-width // 8) * 8        # every segment starts on a 16-byte boundary
+            blocks += [w, w.new_zeros((w.shape[0], padded - width))]
+            self._widths.append((at, width))
+            self._zero_fill |= padded != width
+            at += padded
+        self._joint = Linear(torch.cat(blocks, 1).contiguous())
+        for side in self.sides:
+            side.release_out()
+
     def forward(self, x, batch, cache: CacheView, write: bool, position: PositionEncoding):
+        if self._joint is None:
+            self._join_outputs()
+        if self._joint is not False:
+            w = self._joint.weight
+            # (zeros where segments are padded up to 16 bytes, and in padded steps, whose padding
+            # tokens the attention leaves unwritten)
+            cat = (torch.zeros if self._zero_fill or batch.padded else torch.empty)(
+                (x.shape[0], w.shape[1]), dtype=w.dtype, device=w.device)
+            self.activations_into(x, batch, cache, write, position,
+                                  [cat[:, a:a + n] for a, n in self._widths])
+            return Terms.of(self._joint(cat), self._joint_scale)
         out = None
         for side, scale, view in zip(self.sides, self.scales, self._views(cache)):
             term = Terms.of(side.forward(x, batch, view, write, position), scale)

@@ -114,6 +114,22 @@ class Terms:
         return out
 
 
+@dataclass
+class StreamUpdate:
+    """What a sublayer leaves pending for a residual stream of several parts [tokens, parts, hidden]:
+    ``x_t <- sum_s mix[s, t] x_s + to[t] * y`` with y the sum of ``terms``.  A norm that says
+    ``takes_streams`` carries it out while it reads the parts for the next sublayer."""
+
+    terms: Terms
+    mix: torch.Tensor     # float32 [parts, parts], [from, to]
+    to: torch.Tensor      # float32 [parts]
+
+    def applied(self, parts: torch.Tensor) -> torch.Tensor:
+        """The updated parts as a new tensor, for looking into a model."""
+        y = self.terms.total()
+        return torch.einsum("nsd,st->ntd", parts, self.mix) + self.to[None, :, None] * y[:, None]
+
+
 class StreamSink:
     """Where a branch's last product may put its output: into ``resid``, prepared for ``norm``."""
 
