@@ -218,6 +218,39 @@ def deganex_config(name: str):
         "layers": [state_space, latent, memory, latent]})
 
 
+def kumudra_config(name: str):
+    """The Kumudra design at the sizes of COMPARE_SIZES: two streams; attention (half of the heads,
+    window, biases, a quarter of each head rotated) beside time mixing (heads of 64 across the
+    width) with a dense feed-forward, gated linear attention (keys of 128, values of 256, one head
+    per 256 of the width) and lightning attention (heads of 128 across the width) with a routed
+    one of 16 experts, each a quarter of the dense size, of which a token uses 4, and the two
+    mixers side by side again with a dense one."""
+    from scratch_llm_b200.config import config_from_dict
+
+    z = COMPARE_SIZES[name]
+    d = z["width"]
+    dense = {"kind": "dense", "ff": z["ff"]}
+    routed = {"kind": "moe", "expert": {"ff": z["ff"] // 4},
+              "router": {"experts": 16, "top": 4, "scale": 1.3}}
+    left = {"heads": z["heads"] // 2, "kv_heads": z["kv_heads"] // 2, "dim": z["dim"],
+            "vdim": z["dim"], "scale": z["dim"] ** -0.5, "mask": {"size": z["window"]},
+            "rot": {"base": 500000.0, "dims": z["dim"] // 4,
+                    "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 4096}}}
+    both = {"type": "parallel", "mlp": dense, "mixer": {
+        "left": left, "right": {"heads": d // 64, "dim": 64}, "left_scale": 0.7,
+        "right_scale": 1.1}}
+    gla = {"type": "gla", "mlp": routed, "mixer": {"heads": d // 256, "dim": 128, "vdim": 256,
+                                                   "tau": 16.0}}
+    heads = d // 128
+    lightning = {"type": "lightning", "mlp": routed, "mixer": {
+        "heads": heads, "dim": 128, "vdim": 128,
+        "decay": [1.0 - 2.0 ** (-2.0 - 8.0 * h / heads) for h in range(heads)]}}
+    return config_from_dict({
+        "architecture": "Kumudra", "vocab": z["vocab"], "width": d, "norm": {"eps": 1e-6},
+        "embedding": {"scale": 1.5}, "residual_mult": 0.8, "streams": 2, "max_position": 8192,
+        "layers": [both, gla, lightning, both]})
+
+
 #: low ranks that only a model's tensors say (a size of -1 in a parameter's shape): random
 #: weights are drawn with this one
 RANDOM_LOW_RANK = 64
@@ -256,14 +289,16 @@ def engine_of(cfg, capacity_tokens: int, max_requests: int, page_size: int):
 
 
 def compare_main(args) -> int:
-    """--compare nilevik | vobosun | titedra | tubevik | deganex: prefill and decode throughput of
+    """--compare nilevik | vobosun | titedra | tubevik | deganex | kumudra: prefill and decode throughput of
     that design beside the engine's other models of equal size (for Vobosun: Nilevik, the closest one, a hybrid of
     attention and a delta rule with normed branch outputs, and the Llama-style model; for
     Titedra: Vobosun, the closest one, with norms around every branch, a partly rotated
     attention and routed experts, and the Llama-style model; for Tubevik: Nilevik, the closest one, likewise a hybrid of windowed
     attention and a gated delta rule, and the Llama-style model; for Deganex: Titedra, the closest
     one, with latent attention and routed experts, Nilevik for its recurrence, and the
-    Llama-style model), at the sizes of COMPARE_SIZES.
+    Llama-style model; for Kumudra: Tubevik, the closest one, with attention beside a recurrence
+    with a decay per key channel, Deganex for its scan and routed experts, and the Llama-style
+    model), at the sizes of COMPARE_SIZES.
     One JSON line."""
     import torch
 
@@ -297,6 +332,12 @@ def compare_main(args) -> int:
                 entry["deganex_layers"] = ("state space, latent attention, matrix memory, latent "
                                            "attention, each + routed with a shared expert")
                 archs[:0] = [("deganex", deganex_config(name)), ("titedra", titedra_config(name))]
+            if args.compare == "kumudra":
+                entry["kumudra_layers"] = ("(windowed attention | time mixing) + dense, gated "
+                                           "linear attention + routed, lightning attention + "
+                                           "routed, (windowed attention | time mixing) + dense")
+                archs = [("kumudra", kumudra_config(name)), ("tubevik", tubevik_config(name)),
+                         ("deganex", deganex_config(name))] + [a for a in archs if a[0] == "llama"]
             for arch, cfg in archs:
                 llm = engine_of(cfg, capacity, args.batch + 1, args.page_size)
                 with ClockSampler(0) as clk:
@@ -458,7 +499,8 @@ def main() -> int:
                     help="layer sizes (the default is the configuration the metric is quoted on)")
     ap.add_argument("--serve", type=int, default=0, metavar="N",
                     help="also run the continuous-batching workload with N requests")
-    ap.add_argument("--compare", default=None, choices=["nilevik", "vobosun", "titedra", "tubevik", "deganex"],
+    ap.add_argument("--compare", default=None, choices=["nilevik", "vobosun", "titedra", "tubevik", "deganex",
+                                                        "kumudra"],
                     help="instead of the headline workload: prefill and decode throughput of "
                          "this design beside the Llama-style model of equal size")
     ap.add_argument("--compare-sizes", default=None, choices=sorted(COMPARE_SIZES),
