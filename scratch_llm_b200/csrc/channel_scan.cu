@@ -28,16 +28,18 @@
 // Every exponent is at most 0, however strong the decays: inside blocks of BT = 16 tokens the weights
 // are formed pair by pair and channel by channel; between blocks the exponent is split at the blocks'
 // borders, e^{E_t - start of t's block} * e^{blocks between} * e^{end of s's block - L_s}, whose factors
-// go to q and k beforehand.  Everything is 32-bit fused multiply-adds on the CUDA cores: the operands
-// of every product are 32-bit (decayed keys and queries, the state), and the sizes are small, so the
-// splitting of both operands into bfloat16 parts would cost more than the products.
+// go to q and k beforehand.  In 32-bit, and for the weights in both dtypes, these are fused
+// multiply-adds on the CUDA cores.  The other products of bfloat16 rows run on the tensor cores
+// (mma.sync from shared memory: the contractions are small and need no TMEM accumulator's set-up):
+// what is 32-bit in them (decayed keys and queries, the state, the weights) goes in as three bfloat16
+// parts that hold all of its 24 bits, and where both operands are 32-bit the six products of parts
+// that reach above 2^-24 are formed, all accumulated in 32-bit.
 #include "scan_chunks.cuh"
 
 namespace sllm {
 
 constexpr int BT = 16;              // tokens of a block inside a chunk
 constexpr int NB = TC / BT;
-typedef __nv_bfloat16 bf16;
 
 struct ChannelArgs {
     const void* q; int64_t ldq;          // [tokens, >= H * N]
@@ -51,6 +53,7 @@ struct ChannelArgs {
     float scale;
     int H, N, V;
     int vec4;                            // rows of q, k and log_a allow reads of four elements
+    int vec8;                            // rows of v allow reads of eight elements
     int min_chunked;                     // rows of at least so many tokens are the chunk kernels'
     int n_rows;
     // chunk kernels only
@@ -197,52 +200,85 @@ __device__ __forceinline__ void block_logs(const ChannelArgs& a, const Chunk& c,
         l[i] = (e < a.N && b * BT + i < c.nt) ? lg[(int64_t)i * a.H * a.N] : 0.f;
 }
 
+// Columns [v0, v0 + cols) of the chunk's values into shared memory (bfloat16, row stride ld), zeros
+// beyond V and beyond the chunk's tokens.
+__device__ __forceinline__ void stage_values(const ChannelArgs& a, bf16* dst, int ld, const bf16* v,
+                                             int nt, int v0, int cols) {
+    const int units = cols / 8;
+    for (int i = threadIdx.x; i < TC * units; i += blockDim.x) {
+        const int t = i / units, j = (i - t * units) * 8;
+        alignas(16) bf16 x[8];
+        const bf16* src = v + (int64_t)t * a.ldv + v0 + j;
+        if (t < nt && v0 + j + 8 <= a.V && a.vec8) {
+            *reinterpret_cast<uint4*>(x) = *reinterpret_cast<const uint4*>(src);
+        } else {
+#pragma unroll
+            for (int w = 0; w < 8; ++w)
+                x[w] = t < nt && v0 + j + w < a.V ? src[w] : __float2bfloat16_rn(0.f);
+        }
+        *reinterpret_cast<uint4*>(dst + t * ld + j) = *reinterpret_cast<const uint4*>(x);
+    }
+}
+// The parts of one 32-bit number.
+__device__ __forceinline__ void split1(float x, bf16* part) {
+#pragma unroll
+    for (int p = 0; p < PARTS; ++p) {
+        part[p] = __float2bfloat16_rn(x);
+        x -= __bfloat162float(part[p]);
+    }
+}
+
 // A of one chunk and head; grid (slots, H), 256 threads.  The channels come in slabs of WB.
 constexpr int WB = 64, LDW = WB + 4;
-constexpr int W_FLOATS = 3 * TC * LDW + 2 * NB * WB;
+constexpr int W_FLOATS = 3 * TC * LDW + NB * WB + 3 * WB + WB;
 template <typename T>
-__global__ void __launch_bounds__(256) channel_weights_kernel(const ChannelArgs a) {
+__global__ void __launch_bounds__(256, 3) channel_weights_kernel(const ChannelArgs a) {
     extern __shared__ __align__(16) float sm[];
     float* qs = sm;                       // [TC][LDW]
     float* ks = qs + TC * LDW;            // [TC][LDW]
     float* ps = ks + TC * LDW;            // [TC][LDW]: sums of log_a from the block's start on
     float* tot = ps + TC * LDW;           // [NB][WB]: the blocks' sums
-    float* us = tot + NB * WB;            // [WB]: u (or ones)
+    float* gaps = tot + NB * WB;          // [3][WB]: e^ of block 1's, block 2's, both blocks' sums
+    float* us = gaps + 3 * WB;            // [WB]: u (or ones)
     pdl_wait();
     pdl_trigger();
     Chunk c;
     if (!this_chunk(a, c)) return;
-    const int head = blockIdx.y, tid = threadIdx.x;
+    const int head = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int N = a.N, H = a.H;
     const T* q = reinterpret_cast<const T*>(a.q) + c.n0 * a.ldq + (int64_t)head * N;
     const T* k = reinterpret_cast<const T*>(a.k) + c.n0 * a.ldk + (int64_t)head * N;
-    // within blocks: the strict lower triangles' pairs, two per thread; pair p of a block is (t, s)
-    // with p = t (t - 1) / 2 + s
-    constexpr int PAIRS = BT * (BT - 1) / 2;                 // 120
-    int pt[2], psrc[2];
-    float pair[2] = {0.f, 0.f};
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-        const int p = tid + i * 256, b = p / PAIRS;
-        int r = p - b * PAIRS, t = 1;
+    // Within blocks: tiles of 2 x 2 tokens, 28 below a block's diagonal, two threads a tile (even and
+    // odd quads of channels): threads 0-223.  The tiles on the diagonal have one pair (t, t - 1) with
+    // t odd, one thread each: threads 224-255.
+    const bool single = tid >= 224;
+    int near_t, near_s;                                      // the tile's first tokens
+    if (single) {
+        near_s = (tid - 224) * 2;
+        near_t = near_s;
+    } else {
+        const int blk = tid / 56;
+        int r = (tid - blk * 56) >> 1, t = 1;
         while (r >= t) { r -= t; ++t; }
-        pt[i] = b * BT + t;
-        psrc[i] = b * BT + r;
-        if (b >= NB) pt[i] = -1;
+        near_t = blk * BT + 2 * t;
+        near_s = blk * BT + 2 * r;
     }
-    // between blocks: 64 threads a pair of blocks, 2 x 2 tokens a thread; the six pairs of blocks are
-    // (1,0) (2,1) (3,2) (2,0) and (3,1) (3,0), the second two taken by the first two groups
-    const int group = tid >> 6, in = tid & 63, ti = (in >> 3) * 2, si = (in & 7) * 2;
-    float far[2][4];
+    float near[4] = {0.f, 0.f, 0.f, 0.f};
+    // Between blocks: a warp per pair of blocks, tiles of 4 x 4 tokens, two threads a tile (four quads
+    // of channels each in turn); warps 6 and 7 have the diagonal, a thread per token.
+    const int far_tb = warp < 3 ? warp + 1 : warp == 3 ? 2 : 3;            // (1,0) (2,1) (3,2)
+    const int far_sb = warp < 3 ? warp : warp == 4 ? 1 : 0;                // (2,0) (3,1) (3,0)
+    const float* gap = warp < 3 || warp > 5 ? nullptr : gaps + (warp - 3) * WB;
+    const int far_t = far_tb * BT + (lane >> 3), far_s = far_sb * BT + ((lane >> 1) & 3);
+    float far[4][4];
 #pragma unroll
-    for (int i = 0; i < 2; ++i) far[i][0] = far[i][1] = far[i][2] = far[i][3] = 0.f;
-    const int tb[2] = {group < 3 ? group + 1 : 2, 3};
-    const int sb[2] = {group < 3 ? group : 0, group == 0 ? 1 : 0};
-    float own = 0.f;                                         // the diagonal: four threads a token
+    for (int i = 0; i < 4; ++i) far[i][0] = far[i][1] = far[i][2] = far[i][3] = 0.f;
+    float own = 0.f;
     for (int e0 = 0; e0 < N; e0 += WB) {
         if (e0) __syncthreads();                             // the previous slab is no longer read
-        {   // a thread per (block, channel): 16 tokens
-            const int b = tid / WB, j = tid % WB, e = e0 + j;
+        const int b = tid / WB, j = tid % WB;                // a thread per (block, channel)
+        {
+            const int e = e0 + j;
             float l[BT];
             block_logs(a, c, head, b, e, l);
             float sum = 0.f;
@@ -259,38 +295,58 @@ __global__ void __launch_bounds__(256) channel_weights_kernel(const ChannelArgs 
             if (b == 0) us[j] = !a.u ? 1.f : e < N ? a.u[(int64_t)head * N + e] : 0.f;
         }
         __syncthreads();
-        {   // the diagonal
-            const int t = tid >> 2, part = tid & 3;
+        if (single) {
+            const float* x = qs + (near_t + 1) * LDW;
+            const float* y = ks + near_s * LDW;
+            const float* E = ps + (near_t + (a.u ? 0 : 1)) * LDW;
+            const float* L = ps + near_s * LDW;
+#pragma unroll 4
+            for (int i = 0; i < WB; i += 4) {
+                const float4 xv = load4(x + i), yv = load4(y + i), ev = load4(E + i), lv = load4(L + i);
+                near[2] = fmaf(xv.x * yv.x, __expf(ev.x - lv.x), near[2]);
+                near[2] = fmaf(xv.y * yv.y, __expf(ev.y - lv.y), near[2]);
+                near[2] = fmaf(xv.z * yv.z, __expf(ev.z - lv.z), near[2]);
+                near[2] = fmaf(xv.w * yv.w, __expf(ev.w - lv.w), near[2]);
+            }
+        } else {
+            const float* x = qs + near_t * LDW;
+            const float* y = ks + near_s * LDW;
+            const float* E = ps + (near_t - (a.u ? 1 : 0)) * LDW;
+            const float* L = ps + near_s * LDW;
+#pragma unroll 2
+            for (int i = (tid & 1) * 4; i < WB; i += 8) {
+                float xa[4], xb[4], ya[4], yb[4], ea[4], eb[4], la[4], lb[4];
+                *reinterpret_cast<float4*>(xa) = load4(x + i);
+                *reinterpret_cast<float4*>(xb) = load4(x + LDW + i);
+                *reinterpret_cast<float4*>(ya) = load4(y + i);
+                *reinterpret_cast<float4*>(yb) = load4(y + LDW + i);
+                *reinterpret_cast<float4*>(ea) = load4(E + i);
+                *reinterpret_cast<float4*>(eb) = load4(E + LDW + i);
+                *reinterpret_cast<float4*>(la) = load4(L + i);
+                *reinterpret_cast<float4*>(lb) = load4(L + LDW + i);
 #pragma unroll
-            for (int i = 0; i < WB / 16; ++i) {
-                const int j = (part + 4 * i) * 4;
-                const float4 x = load4(qs + t * LDW + j), y = load4(ks + t * LDW + j), z = load4(us + j);
+                for (int w = 0; w < 4; ++w) {
+                    near[0] = fmaf(xa[w] * ya[w], __expf(ea[w] - la[w]), near[0]);
+                    near[1] = fmaf(xa[w] * yb[w], __expf(ea[w] - lb[w]), near[1]);
+                    near[2] = fmaf(xb[w] * ya[w], __expf(eb[w] - la[w]), near[2]);
+                    near[3] = fmaf(xb[w] * yb[w], __expf(eb[w] - lb[w]), near[3]);
+                }
+            }
+        }
+        if (warp >= 6) {                                     // the diagonal
+            const int t = tid - 192;
+#pragma unroll 4
+            for (int i = 0; i < WB; i += 4) {
+                const float4 x = load4(qs + t * LDW + i), y = load4(ks + t * LDW + i), z = load4(us + i);
                 own = fmaf(x.x * y.x, z.x, fmaf(x.y * y.y, z.y, fmaf(x.z * y.z, z.z,
                       fmaf(x.w * y.w, z.w, own))));
             }
         }
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {                        // pairs of a block
-            if (pt[i] < 0) continue;
-            const float* x = qs + pt[i] * LDW;
-            const float* y = ks + psrc[i] * LDW;
-            const float* Et = ps + (pt[i] - (a.u ? 1 : 0)) * LDW;
-            const float* Ls = ps + psrc[i] * LDW;
-            float acc = pair[i];
-#pragma unroll 4
-            for (int j = 0; j < WB; j += 4) {
-                const float4 xv = load4(x + j), yv = load4(y + j), ev = load4(Et + j), lv = load4(Ls + j);
-                acc = fmaf(xv.x * yv.x, __expf(ev.x - lv.x), acc);
-                acc = fmaf(xv.y * yv.y, __expf(ev.y - lv.y), acc);
-                acc = fmaf(xv.z * yv.z, __expf(ev.z - lv.z), acc);
-                acc = fmaf(xv.w * yv.w, __expf(ev.w - lv.w), acc);
-            }
-            pair[i] = acc;
-        }
         __syncthreads();
         {   // q and k with their factors up to their blocks' borders, in place
-            const int b = tid / WB, j = tid % WB;
             const float end = tot[b * WB + j];
+            if (b > 0)
+                gaps[(b - 1) * WB + j] = expf(b == 3 ? tot[WB + j] + tot[2 * WB + j] : end);
             float before = 0.f;
 #pragma unroll
             for (int i = 0; i < BT; ++i) {
@@ -302,61 +358,61 @@ __global__ void __launch_bounds__(256) channel_weights_kernel(const ChannelArgs 
             }
         }
         __syncthreads();
+        if (warp < 6) {
+            const float* x0 = qs + far_t * LDW;
+            const float* y0 = ks + far_s * LDW;
+#pragma unroll 1
+            for (int i = 0; i < WB / 8; ++i) {
+                const int at = ((i >> 2) * 8 + (lane & 1) * 4 + (i & 3)) * 4;
+                float x[4][4], y[4][4];
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            if (i == 1 && group >= 2) break;
-            const float* x0 = qs + (tb[i] * BT + ti) * LDW;
-            const float* y0 = ks + (sb[i] * BT + si) * LDW;
-            const int gap = tb[i] - sb[i] - 1;               // whole blocks in between
-            float s00 = far[i][0], s01 = far[i][1], s10 = far[i][2], s11 = far[i][3];
-#pragma unroll 4
-            for (int j = 0; j < WB; j += 4) {
-                float xa[4], xb[4], ya[4], yb[4];
-                *reinterpret_cast<float4*>(xa) = load4(x0 + j);
-                *reinterpret_cast<float4*>(xb) = load4(x0 + LDW + j);
-                *reinterpret_cast<float4*>(ya) = load4(y0 + j);
-                *reinterpret_cast<float4*>(yb) = load4(y0 + LDW + j);
-                if (gap > 0) {
+                for (int r = 0; r < 4; ++r) {
+                    *reinterpret_cast<float4*>(x[r]) = load4(x0 + 4 * r * LDW + at);
+                    *reinterpret_cast<float4*>(y[r]) = load4(y0 + 4 * r * LDW + at);
+                }
+                if (gap) {
                     float f[4];
-                    *reinterpret_cast<float4*>(f) = load4(tot + (sb[i] + 1) * WB + j);
-                    if (gap > 1) {
-                        const float4 g = load4(tot + (sb[i] + 2) * WB + j);
-                        f[0] += g.x; f[1] += g.y; f[2] += g.z; f[3] += g.w;
-                    }
+                    *reinterpret_cast<float4*>(f) = load4(gap + at);
 #pragma unroll
-                    for (int w = 0; w < 4; ++w) {
-                        f[w] = __expf(f[w]);
-                        xa[w] *= f[w];
-                        xb[w] *= f[w];
-                    }
+                    for (int r = 0; r < 4; ++r)
+#pragma unroll
+                        for (int w = 0; w < 4; ++w) x[r][w] *= f[w];
                 }
 #pragma unroll
-                for (int w = 0; w < 4; ++w) {
-                    s00 = fmaf(xa[w], ya[w], s00);
-                    s01 = fmaf(xa[w], yb[w], s01);
-                    s10 = fmaf(xb[w], ya[w], s10);
-                    s11 = fmaf(xb[w], yb[w], s11);
-                }
+                for (int r = 0; r < 4; ++r)
+#pragma unroll
+                    for (int s = 0; s < 4; ++s)
+#pragma unroll
+                        for (int w = 0; w < 4; ++w) far[r][s] = fmaf(x[r][w], y[s][w], far[r][s]);
             }
-            far[i][0] = s00; far[i][1] = s01; far[i][2] = s10; far[i][3] = s11;
         }
     }
-    float* A = a.weights + ((int64_t)blockIdx.x * H + head) * TC * TC;
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-        if (pt[i] >= 0) A[pt[i] * TC + psrc[i]] = pair[i];
-        if (i == 1 && group >= 2) continue;
-        float* at = A + (tb[i] * BT + ti) * TC + sb[i] * BT + si;
-        *reinterpret_cast<float2*>(at) = make_float2(far[i][0], far[i][1]);
-        *reinterpret_cast<float2*>(at + TC) = make_float2(far[i][2], far[i][3]);
-    }
-    own += __shfl_xor_sync(0xffffffffu, own, 1);
-    own += __shfl_xor_sync(0xffffffffu, own, 2);
-    if ((tid & 3) == 0) A[(tid >> 2) * TC + (tid >> 2)] = own;
     // (entries above the diagonal are never read)
+    float* A = a.weights + ((int64_t)blockIdx.x * H + head) * TC * TC;
+    if (!single) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) near[i] += __shfl_xor_sync(0xffffffffu, near[i], 1);
+        if ((tid & 1) == 0) {
+            *reinterpret_cast<float2*>(A + near_t * TC + near_s) = make_float2(near[0], near[1]);
+            *reinterpret_cast<float2*>(A + (near_t + 1) * TC + near_s) = make_float2(near[2], near[3]);
+        }
+    } else {
+        A[(near_t + 1) * TC + near_s] = near[2];
+    }
+    if (warp >= 6) {
+        A[(tid - 192) * (TC + 1)] = own;
+    } else {
+#pragma unroll
+        for (int r = 0; r < 4; ++r)
+#pragma unroll
+            for (int s = 0; s < 4; ++s) {
+                const float sum = far[r][s] + __shfl_xor_sync(0xffffffffu, far[r][s], 1);
+                if ((lane & 1) == (s & 1)) A[(far_t + 4 * r) * TC + far_s + 4 * s] = sum;
+            }
+    }
 }
 
-// dS of one chunk and head: a tile of 64 key channels by 64 value columns; grid (slots, H, tiles),
+// dS of one chunk and head (32-bit rows): a tile of 64 key channels by 64 value columns; grid (slots, H, tiles),
 // 128 threads, each 4 channels by 8 columns.
 constexpr int ST_LD = 64 + 4;
 template <typename T>
@@ -477,7 +533,7 @@ __global__ void __launch_bounds__(256) channel_pass_kernel(const ChannelArgs a) 
     *reinterpret_cast<Part*>(home) = S;
 }
 
-// The read-outs of one chunk and head, 64 value columns; grid (slots, H, ceil(V / 64)), 128 threads:
+// The read-outs of one chunk and head (32-bit rows), 64 value columns; grid (slots, H, ceil(V / 64)), 128 threads:
 // thread (tg, vg) has the tokens 8 tg .. 8 tg + 7 and the columns vg, vg + 16, vg + 32, vg + 48.
 constexpr int OB = 32, OLD = OB + 4;                        // channels of a slab
 template <typename T>
@@ -587,22 +643,270 @@ __global__ void __launch_bounds__(128) channel_out_kernel(const ChannelArgs a) {
     }
 }
 
+// dS of one chunk and head on the tensor cores (bfloat16 rows): a tile of 64 key channels by 128 value
+// columns; grid (slots, H, tiles), 256 threads, a warp per 16 columns.
+constexpr int MV = 128, MLD = 64 + 8, MLDV = MV + 8;
+constexpr size_t STATE_MMA_SMEM = ((size_t)PARTS * TC * MLD + (size_t)TC * MLDV) * sizeof(bf16);
+__global__ void __launch_bounds__(256) channel_state_mma_kernel(const ChannelArgs a, int n_tiles) {
+    extern __shared__ __align__(16) unsigned char raw[];
+    __shared__ float tot[NB][64];
+    bf16* ks = reinterpret_cast<bf16*>(raw);               // [PARTS][TC][MLD]: e^{L_last - L_s} k_s
+    bf16* vs = ks + PARTS * TC * MLD;                      // [TC][MLDV]
+    pdl_wait();
+    pdl_trigger();
+    Chunk c;
+    if (!this_chunk(a, c)) return;
+    const int head = blockIdx.y, tid = threadIdx.x;
+    const int N = a.N, V = a.V, H = a.H;
+    const int e0 = (blockIdx.z % n_tiles) * 64, v0 = (blockIdx.z / n_tiles) * MV;
+    const bf16* k = reinterpret_cast<const bf16*>(a.k) + c.n0 * a.ldk + (int64_t)head * N;
+    const bf16* v = reinterpret_cast<const bf16*>(a.v) + c.n0 * a.ldv + (int64_t)head * V;
+    const int j = tid & 63, b = tid >> 6, e = e0 + j;
+    float L[BT];
+    block_logs(a, c, head, b, e, L);
+    bf16 kk[BT];
+#pragma unroll
+    for (int i = 0; i < BT; ++i)
+        kk[i] = (e < N && b * BT + i < c.nt) ? k[(int64_t)(b * BT + i) * a.ldk + e]
+                                             : __float2bfloat16_rn(0.f);
+    stage_values(a, vs, MLDV, v, c.nt, v0, MV);
+#pragma unroll
+    for (int i = 1; i < BT; ++i) L[i] += L[i - 1];
+    const float end = L[BT - 1];
+    tot[b][j] = end;
+    __syncthreads();
+    float after = 0.f;
+    for (int p = NB - 1; p > b; --p) after += tot[p][j];
+#pragma unroll
+    for (int i = 0; i < BT; ++i) {
+        bf16 part[PARTS];
+        split1(__bfloat162float(kk[i]) * expf(after + (end - L[i])), part);
+#pragma unroll
+        for (int p = 0; p < PARTS; ++p) ks[(p * TC + b * BT + i) * MLD + j] = part[p];
+    }
+    if (v0 == 0 && b == 0 && e < N) a.decay[((int64_t)blockIdx.x * H + head) * N + e] = after + end;
+    __syncthreads();
+    const int warp = tid >> 5, lane = tid & 31;
+    if (v0 + warp * 16 >= V) return;
+    // A[m = column][k = token] from [token][column]: transposed 8 x 8 blocks in the order
+    // (m 0-7, k 0-7), (m 8-15, k 0-7), (m 0-7, k 8-15), (m 8-15, k 8-15)
+    uint32_t af[TC / 16][4];
+    const int blk = lane >> 3;
+#pragma unroll
+    for (int kt = 0; kt < TC / 16; ++kt)
+        ldsm4_t(af[kt], smem_addr(vs + (kt * 16 + (blk >> 1) * 8 + (lane & 7)) * MLDV + warp * 16 +
+                                  (blk & 1) * 8));
+    float acc[8][4];
+#pragma unroll
+    for (int u = 0; u < 8; ++u) acc[u][0] = acc[u][1] = acc[u][2] = acc[u][3] = 0.f;
+#pragma unroll
+    for (int p = PARTS - 1; p >= 0; --p)                   // small parts first
+#pragma unroll
+        for (int kt = 0; kt < TC / 16; ++kt)
+#pragma unroll
+            for (int u = 0; u < 8; u += 2) {
+                uint32_t bf[4];
+                ldsm4_t(bf, smem_addr(ks + (p * TC + kt * 16 + (lane & 15)) * MLD + u * 8 +
+                                      (lane >> 4) * 8));
+                mma_bf16(acc[u], af[kt], bf);
+                mma_bf16(acc[u + 1], af[kt], bf + 2);
+            }
+    float* dst = a.dS + ((int64_t)blockIdx.x * H + head) * V * N;
+#pragma unroll
+    for (int u = 0; u < 8; ++u)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            const int m = v0 + warp * 16 + (lane >> 2) + 8 * h, n = e0 + u * 8 + (lane & 3) * 2;
+            if (m >= V || n >= N) continue;
+            float* d = dst + (int64_t)m * N + n;
+            if ((N & 1) == 0) {
+                *reinterpret_cast<float2*>(d) = make_float2(acc[u][2 * h], acc[u][2 * h + 1]);
+            } else {
+                d[0] = acc[u][2 * h];
+                if (n + 1 < N) d[1] = acc[u][2 * h + 1];
+            }
+        }
+}
+
+// The read-outs of one chunk and head on the tensor cores (bfloat16 rows), 64 value columns; grid
+// (slots, H, ceil(V / 64)), 256 threads: warps w and w + 4 have the chunk's tokens 16 w .. 16 w + 15,
+// and half of the columns each.  Queries and state go through shared memory in slabs of 64 channels.
+constexpr size_t OUT_MMA_SMEM = ((size_t)2 * PARTS * TC * MLD + (size_t)TC * MLD) * sizeof(bf16);
+__global__ void __launch_bounds__(256, 3) channel_out_mma_kernel(const ChannelArgs a) {
+    extern __shared__ __align__(16) unsigned char raw[];
+    __shared__ float tot[NB][64];
+    bf16* qs = reinterpret_cast<bf16*>(raw);               // [PARTS][TC][MLD]: e^{E_t} q_t
+    bf16* ss = qs + PARTS * TC * MLD;                      // [PARTS][64][MLD]: S0's columns
+    bf16* vs = ss + PARTS * TC * MLD;                      // [TC][MLD]
+    pdl_wait();
+    pdl_trigger();
+    Chunk c;
+    if (!this_chunk(a, c)) return;
+    const int head = blockIdx.y, v0 = blockIdx.z * 64, tid = threadIdx.x;
+    const int warp = tid >> 5, lane = tid & 31;
+    const int N = a.N, V = a.V, H = a.H;
+    const bf16* q = reinterpret_cast<const bf16*>(a.q) + c.n0 * a.ldq + (int64_t)head * N;
+    const bf16* v = reinterpret_cast<const bf16*>(a.v) + c.n0 * a.ldv + (int64_t)head * V;
+    const float* s0 = a.dS + (((int64_t)blockIdx.x * H + head) * V + v0) * N;
+    stage_values(a, vs, MLD, v, c.nt, v0, 64);
+    const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * 32;
+    float o[4][4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) o[u][0] = o[u][1] = o[u][2] = o[u][3] = 0.f;
+    const int j = tid & 63, b = tid >> 6;
+    for (int e0 = 0; e0 < N; e0 += 64) {
+        const int e = e0 + j;
+        float L[BT];
+        block_logs(a, c, head, b, e, L);
+        bf16 qq[BT];
+#pragma unroll
+        for (int i = 0; i < BT; ++i)
+            qq[i] = (e < N && b * BT + i < c.nt) ? q[(int64_t)(b * BT + i) * a.ldq + e]
+                                                 : __float2bfloat16_rn(0.f);
+        const int se = (tid & 15) * 4;
+        float4 sx[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int col = (tid >> 4) + i * 16;
+            sx[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (v0 + col >= V || e0 + se >= N) continue;
+            const float* at = s0 + (int64_t)col * N + e0 + se;
+            if ((N & 3) == 0) {
+                sx[i] = load4(at);
+            } else {
+                sx[i].x = at[0];
+                if (e0 + se + 1 < N) sx[i].y = at[1];
+                if (e0 + se + 2 < N) sx[i].z = at[2];
+                if (e0 + se + 3 < N) sx[i].w = at[3];
+            }
+        }
+#pragma unroll
+        for (int i = 1; i < BT; ++i) L[i] += L[i - 1];
+        if (e0) __syncthreads();                           // the previous slab is no longer read
+        tot[b][j] = L[BT - 1];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            uint32_t lo[PARTS], hi[PARTS];
+            split2(sx[i].x, sx[i].y, lo);
+            split2(sx[i].z, sx[i].w, hi);
+#pragma unroll
+            for (int p = 0; p < PARTS; ++p)
+                *reinterpret_cast<uint2*>(ss + (p * TC + (tid >> 4) + i * 16) * MLD + se) =
+                    make_uint2(lo[p], hi[p]);
+        }
+        __syncthreads();
+        float before = 0.f;
+        for (int p = 0; p < b; ++p) before += tot[p][j];
+#pragma unroll
+        for (int i = 0; i < BT; ++i) {
+            const float E = before + (a.u ? (i ? L[i - 1] : 0.f) : L[i]);
+            bf16 part[PARTS];
+            split1(__bfloat162float(qq[i]) * expf(E), part);
+#pragma unroll
+            for (int p = 0; p < PARTS; ++p) qs[(p * TC + b * BT + i) * MLD + j] = part[p];
+        }
+        __syncthreads();
+        const int steps = (min(64, N - e0) + 15) / 16;
+        for (int kt = 0; kt < steps; ++kt) {
+            uint32_t af[PARTS][4];
+#pragma unroll
+            for (int p = 0; p < PARTS; ++p)
+                ldsm4(af[p], smem_addr(qs + (p * TC + m0 + (lane & 15)) * MLD + kt * 16 + (lane >> 4) * 8));
+#pragma unroll
+            for (int u = 0; u < 4; u += 2) {
+                uint32_t bf[PARTS][4];
+#pragma unroll
+                for (int p = 0; p < PARTS; ++p)
+                    ldsm4(bf[p], smem_addr(ss + (p * TC + n0 + (u + (lane >> 4)) * 8 + (lane & 7)) * MLD +
+                                           kt * 16 + ((lane >> 3) & 1) * 8));
+#pragma unroll
+                for (int sum = PARTS - 1; sum >= 0; --sum)  // parts p of q and sum - p of S0
+#pragma unroll
+                    for (int p = 0; p <= sum; ++p) {
+                        mma_bf16(o[u], af[p], bf[sum - p]);
+                        mma_bf16(o[u + 1], af[p], bf[sum - p] + 2);
+                    }
+            }
+        }
+    }
+    __syncthreads();
+    // the weights, split, in the queries' place
+    const float* A = a.weights + ((int64_t)blockIdx.x * H + head) * TC * TC;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int t = (tid >> 4) + i * 16, s = (tid & 15) * 4;
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (s <= t) {
+            x = load4(A + t * TC + s);
+            if (s + 1 > t) x.y = 0.f;
+            if (s + 2 > t) x.z = 0.f;
+            if (s + 3 > t) x.w = 0.f;
+        }
+        uint32_t lo[PARTS], hi[PARTS];
+        split2(x.x, x.y, lo);
+        split2(x.z, x.w, hi);
+#pragma unroll
+        for (int p = 0; p < PARTS; ++p)
+            *reinterpret_cast<uint2*>(qs + (p * TC + t) * MLD + s) = make_uint2(lo[p], hi[p]);
+    }
+    __syncthreads();
+    for (int kt = 0; kt * 16 <= m0; ++kt) {                // tokens s of 16
+        uint32_t af[PARTS][4];
+#pragma unroll
+        for (int p = 0; p < PARTS; ++p)
+            ldsm4(af[p], smem_addr(qs + (p * TC + m0 + (lane & 15)) * MLD + kt * 16 + (lane >> 4) * 8));
+#pragma unroll
+        for (int u = 0; u < 4; u += 2) {
+            uint32_t bf[4];
+            ldsm4_t(bf, smem_addr(vs + (kt * 16 + (lane & 15)) * MLD + n0 + u * 8 + (lane >> 4) * 8));
+#pragma unroll
+            for (int p = PARTS - 1; p >= 0; --p) {
+                mma_bf16(o[u], af[p], bf);
+                mma_bf16(o[u + 1], af[p], bf + 2);
+            }
+        }
+    }
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            const int t = m0 + (lane >> 2) + 8 * h, col = v0 + n0 + u * 8 + (lane & 3) * 2;
+            if (t >= c.nt || col >= V) continue;
+            float* d = a.out + (c.n0 + t) * H * V + (int64_t)head * V + col;
+            const float x = o[u][2 * h] * a.scale, y = o[u][2 * h + 1] * a.scale;
+            if ((V & 1) == 0) {
+                *reinterpret_cast<float2*>(d) = make_float2(x, y);
+            } else {
+                d[0] = x;
+                if (col + 1 < V) d[1] = y;
+            }
+        }
+}
+
 template <typename T>
 static cudaError_t launch_chunks(const ChannelArgs& a, int n_tokens, cudaStream_t stream) {
     const int slots = n_tokens / TC + a.n_rows + 1;
     const int nt = (a.N + 63) / 64, vt = (a.V + 63) / 64;
     const size_t smem = (size_t)W_FLOATS * sizeof(float);
+    constexpr bool TENSOR = sizeof(T) == 2;
     static bool ready = false;
     if (!ready) {
-        cudaError_t e = cudaFuncSetAttribute(channel_weights_kernel<T>,
-                                             cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        const cudaFuncAttribute attr = cudaFuncAttributeMaxDynamicSharedMemorySize;
+        cudaError_t e = cudaFuncSetAttribute(channel_weights_kernel<T>, attr, (int)smem);
+        if (e == cudaSuccess && TENSOR)
+            e = cudaFuncSetAttribute(channel_out_mma_kernel, attr, (int)OUT_MMA_SMEM);
         if (e != cudaSuccess) return e;
         ready = true;
     }
     cudaError_t e = sllm_launch_pdl(channel_weights_kernel<T>, dim3(slots, a.H), dim3(256), smem,
                                     stream, a);
     if (e != cudaSuccess) return e;
-    e = sllm_launch_pdl(channel_state_kernel<T>, dim3(slots, a.H, nt * vt), dim3(128), 0, stream, a, nt);
+    if (TENSOR)
+        e = sllm_launch_pdl(channel_state_mma_kernel, dim3(slots, a.H, nt * ((a.V + MV - 1) / MV)),
+                            dim3(256), STATE_MMA_SMEM, stream, a, nt);
+    else
+        e = sllm_launch_pdl(channel_state_kernel<float>, dim3(slots, a.H, nt * vt), dim3(128), 0, stream,
+                            a, nt);
     if (e != cudaSuccess) return e;
     const int64_t size = (int64_t)a.V * a.N;
     if ((a.N & 3) == 0)
@@ -612,7 +916,10 @@ static cudaError_t launch_chunks(const ChannelArgs& a, int n_tokens, cudaStream_
         e = sllm_launch_pdl(channel_pass_kernel<1>, dim3((unsigned)((size + 255) / 256), a.H, a.n_rows),
                             dim3(256), 0, stream, a);
     if (e != cudaSuccess) return e;
-    return sllm_launch_pdl(channel_out_kernel<T>, dim3(slots, a.H, vt), dim3(128), 0, stream, a);
+    if (TENSOR)
+        return sllm_launch_pdl(channel_out_mma_kernel, dim3(slots, a.H, vt), dim3(256), OUT_MMA_SMEM,
+                               stream, a);
+    return sllm_launch_pdl(channel_out_kernel<float>, dim3(slots, a.H, vt), dim3(128), 0, stream, a);
 }
 
 }  // namespace sllm
@@ -638,8 +945,9 @@ SLLM_EXPORT int sllm_channel_scan(const void* q, int64_t ldq, const void* k, int
         return (int)cudaErrorInvalidValue;
     const int vec4 = !((ldq | ldk | N) & 3) &&
                      !(((uintptr_t)q | (uintptr_t)k | (uintptr_t)log_a) & 15);
+    const int vec8 = !((ldv | V) & 7) && !((uintptr_t)v & 15);
     ChannelArgs a = {q, ldq, k, ldk, v, ldv, log_a, u, state, row_start, row_slot, out, scale,
-                     H, N, V, vec4, 0x7fffffff, n_rows, dS, decay, weights};
+                     H, N, V, vec4, vec8, 0x7fffffff, n_rows, dS, decay, weights};
     if ((N & 3) == 0 && ((uintptr_t)state & 15)) return (int)cudaErrorInvalidValue;
     if (chunked) {
         if (!dS || !decay || !weights || min_chunked < 1 ||
