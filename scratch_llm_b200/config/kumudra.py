@@ -33,7 +33,8 @@ config.json::
                 {"type": "lightning", "mixer": {"heads", "dim", "vdim", "decay": [per head]},
                  "mlp": ...}, ...]}
 
-Without ``streams`` the stream is one sum and there are no ``hc`` tensors.
+Without ``streams`` the stream is one sum and there are no ``hc`` tensors; without ``mask`` the
+attention sees every earlier key, without ``rot`` nothing is rotated.
 
 Tensors: ``embed``, ``final.norm`` and per layer i ``l<i>.norm1``, ``l<i>.norm2``,
 ``l<i>.hc1.{in,out,mix}``, ``l<i>.hc2.*``, ``l<i>.mix.*`` (``parallel``: ``l<i>.mix.left.*`` and
@@ -152,8 +153,11 @@ class KumudraConfig:
             raise ValueError(f"{where}: {m['heads']} heads do not group evenly over "
                              f"{m['kv_heads']} key/value heads")
         _number(m.get("scale"), f"{where}.scale")
-        _positive_int(_mapping(m.get("mask"), f"{where}.mask").get("size"), f"{where}.mask.size")
-        rot = _mapping(m.get("rot"), f"{where}.rot")
+        if m.get("mask") is not None:
+            _positive_int(_mapping(m["mask"], f"{where}.mask").get("size"), f"{where}.mask.size")
+        if m.get("rot") is None:
+            return
+        rot = _mapping(m["rot"], f"{where}.rot")
         _positive(rot.get("base"), f"{where}.rot.base")
         dims = _positive_int(rot.get("dims"), f"{where}.rot.dims")
         if dims % 2 or dims > m["dim"]:
@@ -225,23 +229,23 @@ class KumudraConfig:
 
     def _mixer(self, kind: str, m: Mapping[str, Any]) -> tuple[PartSpec, PartSpec]:
         if kind == "parallel":
-            left, right, rot = m["left"], m["right"], m["left"]["rot"]
+            left, right, rot = m["left"], m["right"], m["left"].get("rot")
             attention = {"hidden_size": self.width, "n_heads": left["heads"],
                          "n_kv_heads": left["kv_heads"], "head_dim": left["dim"],
                          "value_dim": left["vdim"], "scale": float(left["scale"]), "bias": True,
-                         "window": left["mask"]["size"],
+                         "window": (left.get("mask") or {}).get("size"),
                          "names": {n: n for n in "qkvo"}}
             time_mixing = {"hidden_size": self.width, "n_heads": right["heads"],
                            "head_dim": right["dim"], "eps": self.norm_eps}
+            position = PartSpec("none") if rot is None else PartSpec("rotary", {
+                "head_dim": left["dim"] + left["dim"] % 2, "theta": float(rot["base"]),
+                "max_position": self.max_position, "interleaved": False,
+                "rot_dims": rot["dims"], "llama3": rot.get("scaling")})
             return (PartSpec("side_by_side", {
                         "left": {"kind": "gqa_attention", "args": attention},
                         "right": {"kind": "time_mixing", "args": time_mixing},
                         "left_scale": float(m["left_scale"]),
-                        "right_scale": float(m["right_scale"])}),
-                    PartSpec("rotary", {
-                        "head_dim": left["dim"] + left["dim"] % 2, "theta": float(rot["base"]),
-                        "max_position": self.max_position, "interleaved": False,
-                        "rot_dims": rot["dims"], "llama3": rot.get("scaling")}))
+                        "right_scale": float(m["right_scale"])}), position)
         common = {"hidden_size": self.width, "n_heads": m["heads"], "key_dim": m["dim"],
                   "value_dim": m["vdim"], "eps": self.norm_eps}
         if kind == "gla":

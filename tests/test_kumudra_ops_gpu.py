@@ -332,7 +332,8 @@ ATTENTION = [  # heads, kv heads, dim, vdim, rot dims, window, page, scaling
     (8, 2, 64, 48, 32, 40, 16, None), (4, 2, 16, 24, 8, 13, 8, (4.0, 1.0, 3.0, 60)),
     (3, 3, 20, 12, 6, 16, 16, None), (2, 1, 128, 128, 128, 65, 32, (8.0, 1.0, 4.0, 400)),
     (4, 1, 64, 64, 16, 128, 64, (2.0, 0.5, 0.5, 100)), (2, 2, 12, 30, 2, 1, 16, None),
-    (6, 3, 32, 64, 32, 500, 16, None)]
+    (6, 3, 32, 64, 32, 500, 16, None), (4, 2, 64, 64, 6, 40, 16, (3.0, 1.0, 2.0, 80)),
+    (2, 2, 60, 64, 22, 33, 16, None), (4, 2, 120, 128, 40, 90, 64, None)]
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
