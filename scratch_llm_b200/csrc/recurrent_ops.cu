@@ -284,6 +284,37 @@ head_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ gate, i
     }
 }
 
+// The same four elements at a time, for heads of up to 128 entries in fours and no divisor: LANES
+// lanes of a warp share a head (a lane has one quad), 128 threads a CTA.
+template <typename T, int LANES>
+__global__ void __launch_bounds__(128)
+head_norm_gate_vec_kernel(const float* __restrict__ o, const T* __restrict__ gate, int64_t ldg,
+                          const float* __restrict__ gain, float eps, T* __restrict__ out, int64_t ldo,
+                          int H, int V, int gain_per_head, int gate_act, int64_t n_heads) {
+    pdl_wait();
+    pdl_trigger();
+    const int64_t idx = (int64_t)blockIdx.x * (128 / LANES) + threadIdx.x / LANES;
+    const int e = (threadIdx.x % LANES) * 4;
+    const bool live = idx < n_heads && e < V;
+    const int64_t n = live ? idx / H : 0;
+    const int head = live ? (int)(idx - n * H) : 0;
+    float v[4] = {0.f, 0.f, 0.f, 0.f}, z[4], gn[4];
+    if (live) {
+        load_few<4>(o + (n * H + head) * V + e, v);
+        load_few<4>(gate + n * ldg + (int64_t)head * V + e, z);
+        load_few<4>(gain + (gain_per_head ? (int64_t)head * V : 0) + e, gn);
+    }
+    float ss = (v[0] * v[0] + v[1] * v[1]) + (v[2] * v[2] + v[3] * v[3]);
+#pragma unroll
+    for (int k = LANES / 2; k > 0; k >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, k);
+    if (!live) return;
+    const float inv = 1.0f / sqrtf(ss / (float)V + eps);
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+        v[k] = v[k] * inv * gn[k] * (gate_act == 1 ? 1.f : z[k]) * sigmoid_of<T>(z[k]);
+    store_few<4>(out + n * ldo + (int64_t)head * V + e, v);
+}
+
 // Decays and removal rates of a delta-rule mixer whose decay comes through a low-rank pair of
 // matrices.  pre: float32 [N, ldp] holds the removal rates' inputs in columns [0, C) and the
 // low-rank hidden values in columns [C, C + R).  w2t: float32 [R, C] (the second matrix,
@@ -355,7 +386,7 @@ lowrank_decay_kernel(const float* __restrict__ pre, int64_t ldp, const float* __
 // The sum runs over r in ascending order for every token, whatever the batch.  out: [N, C],
 // float32 or bfloat16.  One launch serves up to two such products of the same `pre` (a mixer's
 // decays and its gate): the first `blocks0` CTAs along x take the first job, the rest the second.
-// grid (blocks of both jobs, ceil(N / LOWRANK_TOKENS)); shared: LOWRANK_TOKENS * max R floats.
+// grid (blocks of both jobs, ceil(N / TOKENS)); shared: TOKENS * max R floats (R up to a multiple of 4).
 constexpr float LOG_DECAY_FLOOR = -88.f;
 struct ExpandJob {
     int col0; const float* w2t; const float* bias; const float* rate_log; int per_rate; int mode;
@@ -363,47 +394,60 @@ struct ExpandJob {
     void* out; int out_bf16; int C; int R;
 };
 
+// TOKENS of a CTA; its threads' first EXPAND_AHEAD weights are requested before the kernel waits for
+// the ones ahead of it (nothing writes weights).
+constexpr int EXPAND_AHEAD = 16;
+template <int TOKENS>
 __global__ void __launch_bounds__(256)
 lowrank_expand_kernel(const float* __restrict__ pre, int64_t ldp, const ExpandJob j0,
                       const ExpandJob j1, int blocks0, int N) {
-    pdl_wait();
-    pdl_trigger();
-    extern __shared__ float th[];   // [LOWRANK_TOKENS][R]
+    extern __shared__ __align__(16) float th[];   // [TOKENS][RP], zeros from R on
     const bool second = (int)blockIdx.x >= blocks0;
     const ExpandJob& j = second ? j1 : j0;
-    const int R = j.R, C = j.C;
-    const int n0 = blockIdx.y * LOWRANK_TOKENS;
-    const int nt = min(LOWRANK_TOKENS, N - n0);
-    for (int i = threadIdx.x; i < LOWRANK_TOKENS * R; i += blockDim.x) {
-        const int t = i / R, r = i - t * R;
-        const float h = t < nt ? pre[(int64_t)(n0 + t) * ldp + j.col0 + r] : 0.f;
-        th[t * R + r] = j.tanh_in ? tanhf(h) : h;
+    const int R = j.R, C = j.C, RP = (R + 3) / 4 * 4;
+    const int n0 = blockIdx.y * TOKENS;
+    const int nt = min(TOKENS, N - n0);
+    const int c = ((int)blockIdx.x - (second ? blocks0 : 0)) * blockDim.x + threadIdx.x;
+    const float* w2t = j.w2t + (c < C ? c : 0);
+    float w[EXPAND_AHEAD];
+#pragma unroll
+    for (int k = 0; k < EXPAND_AHEAD; ++k) w[k] = k < R ? w2t[(int64_t)k * C] : 0.f;
+    pdl_wait();
+    pdl_trigger();
+    for (int i = threadIdx.x; i < TOKENS * RP; i += blockDim.x) {
+        const int t = i / RP, r = i - t * RP;
+        const float h = t < nt && r < R ? pre[(int64_t)(n0 + t) * ldp + j.col0 + r] : 0.f;
+        th[i] = j.tanh_in ? tanhf(h) : h;
     }
     __syncthreads();
-    const int c = ((int)blockIdx.x - (second ? blocks0 : 0)) * blockDim.x + threadIdx.x;
     if (c >= C) return;
-    float acc[LOWRANK_TOKENS];
+    float acc[TOKENS];
 #pragma unroll
-    for (int t = 0; t < LOWRANK_TOKENS; ++t) acc[t] = 0.f;
-    int r = 0;
-    for (; r + 16 <= R; r += 16) {
-        float w[16];
+    for (int t = 0; t < TOKENS; ++t) acc[t] = 0.f;
+    for (int r = 0; r < R; r += EXPAND_AHEAD) {
+        float next[EXPAND_AHEAD];
 #pragma unroll
-        for (int k = 0; k < 16; ++k) w[k] = j.w2t[(int64_t)(r + k) * C + c];
+        for (int k = 0; k < EXPAND_AHEAD; ++k)
+            next[k] = r + EXPAND_AHEAD + k < R ? w2t[(int64_t)(r + EXPAND_AHEAD + k) * C] : 0.f;
 #pragma unroll
-        for (int k = 0; k < 16; ++k)
+        for (int k = 0; k < EXPAND_AHEAD; k += 4) {
+            if (r + k >= R) break;
 #pragma unroll
-            for (int t = 0; t < LOWRANK_TOKENS; ++t) acc[t] = fmaf(w[k], th[t * R + r + k], acc[t]);
-    }
-    for (; r < R; ++r) {
-        const float w = j.w2t[(int64_t)r * C + c];
+            for (int t = 0; t < TOKENS; ++t) {
+                const float4 h = *reinterpret_cast<const float4*>(th + t * RP + r + k);
+                acc[t] = fmaf(w[k], h.x, acc[t]);
+                acc[t] = fmaf(w[k + 1], h.y, acc[t]);
+                acc[t] = fmaf(w[k + 2], h.z, acc[t]);
+                acc[t] = fmaf(w[k + 3], h.w, acc[t]);
+            }
+        }
 #pragma unroll
-        for (int t = 0; t < LOWRANK_TOKENS; ++t) acc[t] = fmaf(w, th[t * R + r], acc[t]);
+        for (int k = 0; k < EXPAND_AHEAD; ++k) w[k] = next[k];
     }
     const float b0 = j.bias ? j.bias[c] : 0.f;
     const float rate = j.mode == 1 ? expf(j.rate_log[c / j.per_rate]) : 0.f;
 #pragma unroll
-    for (int t = 0; t < LOWRANK_TOKENS; ++t) {
+    for (int t = 0; t < TOKENS; ++t) {
         if (t < nt) {
             float z = acc[t] + b0;
             if (j.mode == 1) z = -rate * (z > 20.f ? z : log1pf(expf(z)));
@@ -718,6 +762,27 @@ SLLM_EXPORT int sllm_head_norm_gate(const float* o, const void* gate, int64_t ld
     dim3 grid(n_tokens, wide ? H : (H + 3) / 4);
     if (H > 65535) return (int)cudaErrorInvalidValue;
     typedef __nv_bfloat16 bf16;
+    if (!den && V % 4 == 0 && V <= 128 && ldg % 4 == 0 && ldo % 4 == 0 &&
+        !(((uintptr_t)o | (uintptr_t)gate | (uintptr_t)gain | (uintptr_t)out) & 15)) {
+        const int64_t heads = (int64_t)n_tokens * H;
+        const int lanes = V <= 16 ? 4 : V <= 32 ? 8 : V <= 64 ? 16 : 32;
+        const unsigned blocks = (unsigned)((heads + 128 / lanes - 1) / (128 / lanes));
+#define SLLM_HNV(T, L)                                                                             \
+    return (int)sllm_launch_pdl(head_norm_gate_vec_kernel<T, L>, dim3(blocks), dim3(128), 0, stream, \
+                                o, (const T*)gate, ldg, gain, eps, (T*)out, ldo, H, V,             \
+                                gain_per_head, gate_act, heads)
+#define SLLM_HNV_T(T)                                                                              \
+    do {                                                                                           \
+        if (lanes == 4) SLLM_HNV(T, 4);                                                            \
+        if (lanes == 8) SLLM_HNV(T, 8);                                                            \
+        if (lanes == 16) SLLM_HNV(T, 16);                                                          \
+        SLLM_HNV(T, 32);                                                                           \
+    } while (0)
+        if (dtype == 0) SLLM_HNV_T(float);
+        if (dtype == 1) SLLM_HNV_T(bf16);
+#undef SLLM_HNV_T
+#undef SLLM_HNV
+    }
 #define SLLM_HNG(T, WIDE)                                                                          \
     head_norm_gate_kernel<T, WIDE><<<grid, 128, 0, stream>>>(o, (const T*)gate, ldg, gain, eps, den, \
                                                              floor, (T*)out, ldo, H, V,            \
@@ -771,16 +836,24 @@ SLLM_EXPORT int sllm_lowrank_expand(const float* pre, int64_t ldp, int n_jobs, c
         max_r = R[i] > max_r ? R[i] : max_r;
         max_c = C[i] > max_c ? C[i] : max_c;
     }
-    // steps of few tokens: narrow CTAs, so that the channels spread over more SMs
+    // steps of few tokens: narrow CTAs, so that the channels spread over more SMs; long steps: more
+    // tokens a CTA, so that the weights are read less often
     const int threads = n_tokens <= 2 * LOWRANK_TOKENS && max_c >= 1024 ? 64 : 256;
+    const int tokens = n_tokens >= 512 ? 2 * LOWRANK_TOKENS : LOWRANK_TOKENS;
     const int blocks0 = (j[0].C + threads - 1) / threads;
     const int blocks1 = n_jobs > 1 ? (j[1].C + threads - 1) / threads : 0;
-    dim3 grid(blocks0 + blocks1, (n_tokens + LOWRANK_TOKENS - 1) / LOWRANK_TOKENS);
+    dim3 grid(blocks0 + blocks1, (n_tokens + tokens - 1) / tokens);
+    const size_t smem = (size_t)tokens * ((max_r + 3) / 4 * 4) * sizeof(float);
     if (grid.y > 65535) return (int)cudaErrorInvalidValue;
-    lowrank_expand_kernel<<<grid, threads, LOWRANK_TOKENS * max_r * sizeof(float), stream>>>(
-        pre, ldp, j[0], j[1], blocks0, n_tokens);
-    SLLM_LAUNCH_CHECK();
-    return 0;
+    if (smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(lowrank_expand_kernel<2 * LOWRANK_TOKENS>,
+                                             cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+    }
+    return (int)sllm_launch_pdl(tokens == LOWRANK_TOKENS ? lowrank_expand_kernel<LOWRANK_TOKENS>
+                                                         : lowrank_expand_kernel<2 * LOWRANK_TOKENS>,
+                                grid, dim3(threads), smem, stream, pre, ldp, j[0], j[1], blocks0,
+                                n_tokens);
 }
 
 // out = parts of o * act(gate) over their root mean squares, times gain; after: parts of o over
