@@ -104,18 +104,18 @@ __global__ void __launch_bounds__(256) gated_scan_kernel(const ScanArgs a, int t
             for (int w = 0; w < 4; ++w) S[4 * i + w] = (live && e + w < N) ? st[e + w] : 0.f;
         }
     }
-    if (n_new == 1 && quads && a.vec4) {       // decoding: nothing is staged
+    // decoding: nothing is staged (with a silu it is: every column's lanes would form it again)
+    if (n_new == 1 && quads && a.vec4 && !a.silu) {
         const int64_t n = t0;
         const float decay = expf(a.log_a[n * a.ld_gates + head]);
-        const float value = !is_ones ? silu_if(to_float(v[n * a.ldv + col]), a.silu) : 1.f;
+        const float value = !is_ones ? to_float(v[n * a.ldv + col]) : 1.f;
         const float bv = a.b ? a.b[n * H + head] * value : value;
         float acc = 0.f;
 #pragma unroll
         for (int i = 0; i < QPL; ++i) {
             const int e = (i * LPC + sub) * 4;
             if (e < N) {
-                const float4 kk = silu_if(load4(k + n * a.ldk + e), a.silu);
-                const float4 qq = silu_if(load4(q + n * a.ldq + e), a.silu);
+                const float4 kk = load4(k + n * a.ldk + e), qq = load4(q + n * a.ldq + e);
                 float4 x;
                 x.x = fmaf(decay, S[4 * i], bv * kk.x);
                 x.y = fmaf(decay, S[4 * i + 1], bv * kk.y);

@@ -394,24 +394,27 @@ struct ExpandJob {
     void* out; int out_bf16; int C; int R;
 };
 
-// TOKENS of a CTA; its threads' first EXPAND_AHEAD weights are requested before the kernel waits for
-// the ones ahead of it (nothing writes weights).
-constexpr int EXPAND_AHEAD = 16;
-template <int TOKENS>
+// A CTA has TOKENS tokens and CH channels a thread (2: C even); a thread's next AHEAD rows of
+// weights are in flight while it works on the ones before, the first ones already before the kernel
+// waits for those ahead of it (nothing writes weights).
+template <int TOKENS, int CH, int AHEAD>
 __global__ void __launch_bounds__(256)
 lowrank_expand_kernel(const float* __restrict__ pre, int64_t ldp, const ExpandJob j0,
                       const ExpandJob j1, int blocks0, int N) {
     extern __shared__ __align__(16) float th[];   // [TOKENS][RP], zeros from R on
+    struct alignas(4 * CH) Weights { float x[CH]; };
     const bool second = (int)blockIdx.x >= blocks0;
     const ExpandJob& j = second ? j1 : j0;
     const int R = j.R, C = j.C, RP = (R + 3) / 4 * 4;
     const int n0 = blockIdx.y * TOKENS;
     const int nt = min(TOKENS, N - n0);
-    const int c = ((int)blockIdx.x - (second ? blocks0 : 0)) * blockDim.x + threadIdx.x;
+    const int c = (((int)blockIdx.x - (second ? blocks0 : 0)) * blockDim.x + threadIdx.x) * CH;
     const float* w2t = j.w2t + (c < C ? c : 0);
-    float w[EXPAND_AHEAD];
+    const Weights none = {};
+    Weights w[AHEAD];
 #pragma unroll
-    for (int k = 0; k < EXPAND_AHEAD; ++k) w[k] = k < R ? w2t[(int64_t)k * C] : 0.f;
+    for (int k = 0; k < AHEAD; ++k)
+        w[k] = k < R ? *reinterpret_cast<const Weights*>(w2t + (int64_t)k * C) : none;
     pdl_wait();
     pdl_trigger();
     for (int i = threadIdx.x; i < TOKENS * RP; i += blockDim.x) {
@@ -421,42 +424,61 @@ lowrank_expand_kernel(const float* __restrict__ pre, int64_t ldp, const ExpandJo
     }
     __syncthreads();
     if (c >= C) return;
-    float acc[TOKENS];
+    float acc[TOKENS][CH];
 #pragma unroll
-    for (int t = 0; t < TOKENS; ++t) acc[t] = 0.f;
-    for (int r = 0; r < R; r += EXPAND_AHEAD) {
-        float next[EXPAND_AHEAD];
+    for (int t = 0; t < TOKENS; ++t)
 #pragma unroll
-        for (int k = 0; k < EXPAND_AHEAD; ++k)
-            next[k] = r + EXPAND_AHEAD + k < R ? w2t[(int64_t)(r + EXPAND_AHEAD + k) * C] : 0.f;
+        for (int h = 0; h < CH; ++h) acc[t][h] = 0.f;
+    for (int r = 0; r < R; r += AHEAD) {
+        Weights next[AHEAD];
 #pragma unroll
-        for (int k = 0; k < EXPAND_AHEAD; k += 4) {
+        for (int k = 0; k < AHEAD; ++k)
+            next[k] = r + AHEAD + k < R
+                ? *reinterpret_cast<const Weights*>(w2t + (int64_t)(r + AHEAD + k) * C) : none;
+#pragma unroll
+        for (int k = 0; k < AHEAD; k += 4) {
             if (r + k >= R) break;
 #pragma unroll
             for (int t = 0; t < TOKENS; ++t) {
-                const float4 h = *reinterpret_cast<const float4*>(th + t * RP + r + k);
-                acc[t] = fmaf(w[k], h.x, acc[t]);
-                acc[t] = fmaf(w[k + 1], h.y, acc[t]);
-                acc[t] = fmaf(w[k + 2], h.z, acc[t]);
-                acc[t] = fmaf(w[k + 3], h.w, acc[t]);
+                float x[4];
+                *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(th + t * RP + r + k);
+#pragma unroll
+                for (int u = 0; u < 4; ++u)
+#pragma unroll
+                    for (int h = 0; h < CH; ++h) acc[t][h] = fmaf(w[k + u].x[h], x[u], acc[t][h]);
             }
         }
 #pragma unroll
-        for (int k = 0; k < EXPAND_AHEAD; ++k) w[k] = next[k];
+        for (int k = 0; k < AHEAD; ++k) w[k] = next[k];
     }
-    const float b0 = j.bias ? j.bias[c] : 0.f;
-    const float rate = j.mode == 1 ? expf(j.rate_log[c / j.per_rate]) : 0.f;
+    float b0[CH], rate[CH];
+#pragma unroll
+    for (int h = 0; h < CH; ++h) {
+        b0[h] = j.bias ? j.bias[c + h] : 0.f;
+        rate[h] = j.mode == 1 ? expf(j.rate_log[(c + h) / j.per_rate]) : 0.f;
+    }
 #pragma unroll
     for (int t = 0; t < TOKENS; ++t) {
-        if (t < nt) {
-            float z = acc[t] + b0;
-            if (j.mode == 1) z = -rate * (z > 20.f ? z : log1pf(expf(z)));
+        if (t >= nt) break;
+#pragma unroll
+        for (int h = 0; h < CH; ++h) {
+            float z = acc[t][h] + b0[h];
+            if (j.mode == 1) z = -rate[h] * (z > 20.f ? z : log1pf(expf(z)));
             else if (j.mode == 2)
                 z = fmaxf(j.rate * (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))), LOG_DECAY_FLOOR);
             else if (j.mode == 3) z = fmaxf(-expf(z), LOG_DECAY_FLOOR);
-            const int64_t at = (int64_t)(n0 + t) * C + c;
-            if (j.out_bf16) reinterpret_cast<__nv_bfloat16*>(j.out)[at] = __float2bfloat16_rn(z);
-            else reinterpret_cast<float*>(j.out)[at] = z;
+            acc[t][h] = z;
+        }
+        const int64_t at = (int64_t)(n0 + t) * C + c;
+        if (j.out_bf16) {
+#pragma unroll
+            for (int h = 0; h < CH; ++h)
+                reinterpret_cast<__nv_bfloat16*>(j.out)[at + h] = __float2bfloat16_rn(acc[t][h]);
+        } else {
+            Weights out;
+#pragma unroll
+            for (int h = 0; h < CH; ++h) out.x[h] = acc[t][h];
+            *reinterpret_cast<Weights*>(reinterpret_cast<float*>(j.out) + at) = out;
         }
     }
 }
@@ -837,23 +859,27 @@ SLLM_EXPORT int sllm_lowrank_expand(const float* pre, int64_t ldp, int n_jobs, c
         max_c = C[i] > max_c ? C[i] : max_c;
     }
     // steps of few tokens: narrow CTAs, so that the channels spread over more SMs; long steps: more
-    // tokens a CTA, so that the weights are read less often
-    const int threads = n_tokens <= 2 * LOWRANK_TOKENS && max_c >= 1024 ? 64 : 256;
-    const int tokens = n_tokens >= 512 ? 2 * LOWRANK_TOKENS : LOWRANK_TOKENS;
-    const int blocks0 = (j[0].C + threads - 1) / threads;
-    const int blocks1 = n_jobs > 1 ? (j[1].C + threads - 1) / threads : 0;
+    // tokens a CTA and two channels a thread, so that the weights are read less often
+    bool wide = n_tokens >= 512;
+    for (int i = 0; i < n_jobs; ++i)
+        wide = wide && C[i] % 2 == 0 && !(((uintptr_t)w2t[i] | (uintptr_t)out[i]) & 7);
+    const int tokens = wide ? 2 * LOWRANK_TOKENS : LOWRANK_TOKENS;
+    const int threads = wide ? 128 : n_tokens <= 2 * LOWRANK_TOKENS && max_c >= 1024 ? 64 : 256;
+    const int channels = wide ? 2 * threads : threads;
+    const int blocks0 = (j[0].C + channels - 1) / channels;
+    const int blocks1 = n_jobs > 1 ? (j[1].C + channels - 1) / channels : 0;
     dim3 grid(blocks0 + blocks1, (n_tokens + tokens - 1) / tokens);
     const size_t smem = (size_t)tokens * ((max_r + 3) / 4 * 4) * sizeof(float);
     if (grid.y > 65535) return (int)cudaErrorInvalidValue;
+    auto kernel = wide ? lowrank_expand_kernel<2 * LOWRANK_TOKENS, 2, 8>
+                       : lowrank_expand_kernel<LOWRANK_TOKENS, 1, 16>;
     if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(lowrank_expand_kernel<2 * LOWRANK_TOKENS>,
-                                             cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                             (int)smem);
         if (e != cudaSuccess) return (int)e;
     }
-    return (int)sllm_launch_pdl(tokens == LOWRANK_TOKENS ? lowrank_expand_kernel<LOWRANK_TOKENS>
-                                                         : lowrank_expand_kernel<2 * LOWRANK_TOKENS>,
-                                grid, dim3(threads), smem, stream, pre, ldp, j[0], j[1], blocks0,
-                                n_tokens);
+    return (int)sllm_launch_pdl(kernel, grid, dim3(threads), smem, stream, pre, ldp, j[0], j[1],
+                                blocks0, n_tokens);
 }
 
 // out = parts of o * act(gate) over their root mean squares, times gain; after: parts of o over

@@ -265,10 +265,10 @@ def test_token_shift_leaves_padding_alone():
     assert not torch.isnan(out).any()
 
 
-@pytest.mark.parametrize("R, C", [(1, 5), (16, 96), (37, 300), (64, 1024)])
-def test_log_decays_through_a_low_rank_pair(R, C):
+@pytest.mark.parametrize("n", [1, 19, 530])
+@pytest.mark.parametrize("R, C", [(1, 5), (16, 96), (37, 300), (64, 1024), (130, 258)])
+def test_log_decays_through_a_low_rank_pair(R, C, n):
     g, rnd = rnd_of(R)
-    n = 19
     pre, w2t, bias = rnd(n, R + 3, std=2.0), rnd(R, C, std=R ** -0.5), rnd(C, std=6.0)
     bias[0], bias[1] = 200.0, -200.0                  # beyond both ends
     hidden = pre[:, 2:2 + R].double()
