@@ -39,7 +39,7 @@ def draw_layer(rng):
                            mlp=draw_mlp(rng))
     # (a few head sizes, so that the attention kernels are compiled for few)
     top = rng.choice([16, 32, 48, 64, 128])
-    dim, vdim = top - rng.randint(0, 15), rng.randint(1, top)
+    dim, vdim = max(2, top - rng.randint(0, 15)), rng.randint(1, top)
     if rng.random() < 0.5 and vdim >= 2:
         dim, vdim = max(2, vdim), dim
     kv = rng.choice([1, 2, 3])
